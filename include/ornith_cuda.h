@@ -320,6 +320,24 @@ int32_t orn_model_init_random(orn_model* m, uint64_t seed);
 /* TextModel::load + MtpHead::load (src/weights.rs:41-279): safetensors shards
  * + config.json in `dir`; mtp sidecar if present */
 int32_t orn_model_load(orn_ctx* ctx, const char* dir, int32_t max_ctx, orn_model** out);
+/* The same with the activation type stated.  config.json chooses the architecture: its "architecture"
+ * names an entry of the model registry ("Peratar"); without one it is the Qwen3.5-MoE trunk (bfloat16
+ * only).  ORN_DT_F32 runs everything in true float32 (bf16 weights, float32 activations and caches). */
+#define ORN_DT_BF16 0
+#define ORN_DT_F32 1
+int32_t orn_model_load_as(orn_ctx* ctx, const char* dir, int32_t max_ctx, int32_t dtype, orn_model** out);
+/* a registered architecture from the text of a config.json, without weights (orn_model_init_random or
+ * orn_model_set_linear / orn_model_set_tensor supply them) */
+int32_t orn_model_create_json(orn_ctx* ctx, const char* config_json, int32_t max_ctx, int32_t dtype, orn_model** out);
+/* Run n tokens from the cache's position (chunks of prefill_step rows, windows of up to 4 rows) and
+ * advance it; dev_logits [n_want, vocab] float32 receives the logits at the ascending places host_want[]
+ * among these tokens (n_want may be 0).  Serves every architecture of the registry. */
+int32_t orn_step(orn_model* m, orn_cache* c, const uint32_t* host_ids, int32_t n, int32_t prefill_step,
+                 const int32_t* host_want, int32_t n_want, float* dev_logits);
+/* a checker's view of the layers: during every later orn_step of n tokens dev_tap [layers, n, hidden]
+ * receives the float32 stream after each layer (NULL: off).  Registered decoders only; windows then run
+ * without CUDA graphs. */
+int32_t orn_model_tap(orn_model* m, float* dev_tap);
 /* look a weight up again (checkers export it for the CPU oracle) */
 int32_t orn_model_get_linear(orn_model* m, const char* name, const orn_linear** out);
 int32_t orn_model_get_tensor(orn_model* m, const char* name, const uint16_t** dev_out, size_t* n);
@@ -333,7 +351,8 @@ int32_t orn_cache_create(orn_model* m, orn_cache** out);     /* make_cache + mak
 int32_t orn_cache_destroy(orn_cache* c);
 int32_t orn_cache_reset(orn_cache* c);
 int32_t orn_cache_offset(const orn_cache* c);
-/* TextModel::forward_hidden: T <= 4 rows per call; dev_normed [T,H] */
+/* TextModel::forward_hidden: T <= 4 rows per call; dev_normed [T,H].  Row buffers of every call are in
+ * the model's activation type, a hidden row padded to a multiple of 8 elements. */
 int32_t orn_forward(orn_model* m, orn_cache* c, const uint32_t* host_ids, int32_t T,
                     uint16_t* dev_normed, uint16_t* dev_pre_norm /*nullable*/);
 /* generate::prefill (src/generate.rs:90-136) over all n tokens: chunks of prefill_step rows

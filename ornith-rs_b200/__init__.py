@@ -12,15 +12,16 @@ Activations are bfloat16 carried as numpy uint16; device buffers are `DevBuf`.
 There is no CPU fallback: every call runs a CUDA kernel or raises.
 """
 import ctypes as C
+import json
 
 import numpy as np
 
 from . import _ffi
-from ._ffi import A4, A8, BF16, POLICY_COMMITTED, POLICY_CYCLE, Q4K, Q6K, Config, ForceDraft, MtpStats, Prof
+from ._ffi import A4, A8, BF16, DT_BF16, DT_F32, POLICY_COMMITTED, POLICY_CYCLE, Q4K, Q6K, Config, ForceDraft, MtpStats, Prof
 
 __all__ = [
     "Context", "DevBuf", "Linear", "TextModel", "Cache", "Config", "MtpStats", "OrnError",
-    "Q4K", "Q6K", "A8", "BF16", "A4", "POLICY_CYCLE", "POLICY_COMMITTED", "generate_step",
+    "Q4K", "Q6K", "A8", "BF16", "A4", "POLICY_CYCLE", "POLICY_COMMITTED", "DT_BF16", "DT_F32", "generate_step",
     "generate_step_mtp", "qwen35_config", "lib",
 ]
 
@@ -245,19 +246,36 @@ class TextModel:
 
     def __init__(self, ctx, cfg):
         self.ctx, self.cfg = ctx, cfg
+        self.act, self.logit, self.row_elems = np.uint16, np.uint16, cfg.hidden
         h = C.c_void_p()
         ctx.check(ctx._lib.orn_model_create(ctx.h, C.byref(cfg), C.byref(h)), "orn_model_create")
         self.h = h
 
     @classmethod
-    def load(cls, ctx, directory, max_ctx=512):
-        """TextModel::load + MtpHead::load from safetensors shards (src/weights.rs:41-279)."""
+    def load(cls, ctx, directory, max_ctx=512, dtype=DT_BF16):
+        """TextModel::load + MtpHead::load from safetensors shards (src/weights.rs:41-279); config.json
+        chooses the architecture, dtype the activation type (DT_F32: architectures that run in it)."""
         h = C.c_void_p()
-        ctx.check(ctx._lib.orn_model_load(ctx.h, directory.encode(), max_ctx, C.byref(h)), "orn_model_load")
+        ctx.check(ctx._lib.orn_model_load_as(ctx.h, directory.encode(), max_ctx, dtype, C.byref(h)), "orn_model_load_as")
+        return cls._adopt(ctx, h, dtype)
+
+    @classmethod
+    def from_config(cls, ctx, config, max_ctx=512, dtype=DT_BF16):
+        """A registered architecture from its config.json (a dict), without weights."""
+        h = C.c_void_p()
+        ctx.check(ctx._lib.orn_model_create_json(ctx.h, json.dumps(config).encode(), max_ctx, dtype, C.byref(h)),
+                  "orn_model_create_json")
+        return cls._adopt(ctx, h, dtype)
+
+    @classmethod
+    def _adopt(cls, ctx, h, dtype):
         self = cls.__new__(cls)
         self.ctx, self.h = ctx, h
         self.cfg = Config()
         ctx.check(ctx._lib.orn_model_config(h, C.byref(self.cfg)), "orn_model_config")
+        self.act = np.float32 if dtype == DT_F32 else np.uint16
+        self.row_elems = -(-self.cfg.hidden // 8) * 8
+        self.logit = np.uint16 if self.cfg.n_heads else np.float32  # registered decoders: float32 logits
         return self
 
     def init_random(self, seed):
@@ -304,7 +322,7 @@ class TextModel:
         """forward_hidden / forward_capture: returns the post-norm hidden rows (device)."""
         ids = np.ascontiguousarray(ids, np.uint32)
         T = len(ids)
-        out = self.ctx.empty((T, self.cfg.hidden), np.uint16)
+        out = self.ctx.empty((T, self.row_elems), self.act)
         if capture:
             rc = self.ctx._lib.orn_forward_capture(self.h, cache.h, ids.ctypes.data, T, out.ptr)
         else:
@@ -316,10 +334,35 @@ class TextModel:
         """generate::prefill over all ids; chunks of 64 rows or more run on the tensor cores.
         want_hidden: returns the post-norm hidden rows [n, hidden] (device)."""
         ids = np.ascontiguousarray(ids, np.uint32)
-        out = self.ctx.empty((len(ids), self.cfg.hidden), np.uint16) if want_hidden else None
+        out = self.ctx.empty((len(ids), self.row_elems), self.act) if want_hidden else None
         self.ctx.check(self.ctx._lib.orn_prefill(self.h, cache.h, ids.ctypes.data, len(ids), prefill_step, _p(out)),
                        "orn_prefill")
         return out
+
+    def step(self, cache, ids, want=(), prefill_step=8192):
+        """Run ids from the cache's position; returns the float32 logits [len(want), vocab] at the
+        ascending places `want` among them (numpy)."""
+        ids = np.ascontiguousarray(ids, np.uint32)
+        want = np.ascontiguousarray(want, np.int32)
+        out = self.ctx.empty((len(want), self.cfg.vocab), np.float32) if len(want) else None
+        try:
+            self.ctx.check(self.ctx._lib.orn_step(self.h, cache.h, ids.ctypes.data, len(ids), prefill_step,
+                                                  want.ctypes.data, len(want), _p(out)), "orn_step")
+            return out.numpy() if out is not None else np.empty((0, self.cfg.vocab), np.float32)
+        finally:
+            if out is not None:
+                out.free()
+
+    def step_layers(self, cache, ids, prefill_step=8192):
+        """The float32 stream after every layer while ids run: [layers, len(ids), hidden] (numpy)."""
+        tap = self.ctx.zeros((self.cfg.n_layers, len(ids), self.cfg.hidden), np.float32)
+        self.ctx.check(self.ctx._lib.orn_model_tap(self.h, tap.ptr), "orn_model_tap")
+        try:
+            self.step(cache, ids, prefill_step=prefill_step)
+            return tap.numpy()
+        finally:
+            self.ctx._lib.orn_model_tap(self.h, None)
+            tap.free()
 
     def mtp_forward(self, cache, hidden, ids, kv_only=False):
         """MtpHead::forward for len(ids) rows; returns the draft (raw-logit argmax of the last row) or None."""
@@ -331,7 +374,7 @@ class TextModel:
 
     def head_greedy(self, hidden, T, want_logits=False):
         toks = np.zeros(T, np.uint32)
-        logits = self.ctx.empty((T, self.cfg.vocab), np.uint16) if want_logits else None
+        logits = self.ctx.empty((T, self.cfg.vocab), self.logit) if want_logits else None
         self.ctx.check(self.ctx._lib.orn_head_greedy(self.h, _p(hidden), T, toks.ctypes.data, _p(logits)),
                        "orn_head_greedy")
         return (toks, logits) if want_logits else toks

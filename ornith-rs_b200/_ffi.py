@@ -11,6 +11,7 @@ LIB_PATH = os.environ.get("ORN_CUDA_LIB") or os.path.join(_HERE, "libornith_cuda
 
 Q4K, Q6K, A8, BF16, A4 = 0, 1, 2, 3, 4
 POLICY_CYCLE, POLICY_COMMITTED = 0, 1
+DT_BF16, DT_F32 = 0, 1
 
 c_void_pp = C.POINTER(C.c_void_p)
 u16p = C.c_void_p
@@ -124,6 +125,10 @@ SIGNATURES = {
     "orn_model_set_tensor": (i32, [vp, C.c_char_p, vp, sz]),
     "orn_model_init_random": (i32, [vp, u64]),
     "orn_model_load": (i32, [vp, C.c_char_p, i32, c_void_pp]),
+    "orn_model_load_as": (i32, [vp, C.c_char_p, i32, i32, c_void_pp]),
+    "orn_model_create_json": (i32, [vp, C.c_char_p, i32, i32, c_void_pp]),
+    "orn_step": (i32, [vp, vp, vp, i32, i32, vp, i32, vp]),
+    "orn_model_tap": (i32, [vp, vp]),
     "orn_model_get_linear": (i32, [vp, C.c_char_p, c_void_pp]),
     "orn_model_get_tensor": (i32, [vp, C.c_char_p, c_void_pp, C.POINTER(sz)]),
     "orn_model_config": (i32, [vp, C.POINTER(Config)]),

@@ -14,7 +14,8 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(HERE, "build")
 LIB = os.path.join(HERE, "libornith_cuda.so")
-SOURCES = ["api.cu", "linear.cu", "ops.cu", "gdn.cu", "attn.cu", "sample.cu", "model.cu", "loader.cu", "fused.cu", "gemm.cu", "ep.cu", "batch.cu", "flash.cu", "gdn_chunk.cu"]
+SOURCES = ["api.cu", "linear.cu", "ops.cu", "gdn.cu", "attn.cu", "sample.cu", "model.cu", "loader.cu", "fused.cu", "gemm.cu", "ep.cu", "batch.cu", "flash.cu", "gdn_chunk.cu",
+           "decoder.cu", "dense.cu", "latent.cu"]
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -43,7 +44,17 @@ def _compile(src, verbose):
     return obj, r.stderr
 
 
+def _up_to_date():
+    """The library is newer than everything it is made from (it may have travelled without its objects)."""
+    if not os.path.exists(LIB):
+        return False
+    newest = max([os.path.getmtime(os.path.join(CSRC, s)) for s in SOURCES] + [os.path.getmtime(os.path.abspath(__file__)), _newest_header()])
+    return os.path.getmtime(LIB) > newest
+
+
 def build(verbose=False):
+    if _up_to_date():
+        return LIB
     os.makedirs(OBJ, exist_ok=True)
     with ThreadPoolExecutor(max_workers=8) as ex:
         results = list(ex.map(lambda s: _compile(s, verbose), SOURCES))
@@ -52,7 +63,7 @@ def build(verbose=False):
     if log:
         with open(os.path.join(OBJ, "ptxas.log"), "a") as f:
             f.write(log)
-    if (not os.path.exists(LIB)) or any(os.path.getmtime(o) > os.path.getmtime(LIB) for o in objs):
+    if not _up_to_date():
         cmd = [NVCC, "-shared", "-o", LIB] + objs + ["-lcudart", "-ldl"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:

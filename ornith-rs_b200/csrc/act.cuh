@@ -1,0 +1,32 @@
+// Activations that kernels apply to a float32 product before it is stored.
+#pragma once
+
+#include "orn_common.cuh"
+
+enum { ACT_NONE = 0, ACT_XIELU = 1, ACT_SOFTCAP = 2 };
+
+// xIELU with the two learned numbers (p, q): a = softplus(p) scales the square above zero,
+// b = 1/2 + softplus(q) the exponential below; the slope at zero is 1/2 on both sides.
+struct ActParams {
+  int kind = ACT_NONE;
+  const bf16_t* pq = nullptr;  // ACT_XIELU: device array of two
+  float cap = 0.f;             // ACT_SOFTCAP: cap * tanh(z / cap)
+};
+
+#ifdef __CUDACC__
+ORN_D float act_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+// the two scalars an activation needs, once per thread
+ORN_D void act_prepare(const ActParams& A, float& a, float& b) {
+  a = A.cap; b = 0.f;
+  if (A.kind == ACT_XIELU) {
+    a = act_softplus(bf2f(A.pq[0]));
+    b = 0.5f + act_softplus(bf2f(A.pq[1]));
+  }
+}
+ORN_D float act_apply(int kind, float z, float a, float b) {
+  if (kind == ACT_XIELU) return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, expm1f(z) - z, 0.5f * z);
+  if (kind == ACT_SOFTCAP) return a * tanhf(z / a);
+  return z;
+}
+ORN_D float sigmoid_f32(float z) { return 1.0f / (1.0f + expf(-z)); }
+#endif

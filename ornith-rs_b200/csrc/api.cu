@@ -430,6 +430,7 @@ int32_t orn_gather_gemv(orn_ctx* ctx, const orn_linear* lin, const uint16_t* dev
 
 int32_t orn_gemm(orn_ctx* ctx, const orn_linear* lin, const uint16_t* dev_x, int32_t M, void* dev_y, int32_t out_f32) {
   if (!ctx || !lin || !dev_x || !dev_y || M < 1) return ORN_ERR_ARG;
+  if (lin->K % 64) ORN_FAIL(ctx, ORN_ERR_ARG, "gemm: K must be a multiple of 64");
   return f_qgemm(ctx, ctx->stream, lin, dev_x, M, dev_y, lin->O, nullptr, nullptr, out_f32);
 }
 
@@ -439,6 +440,7 @@ int32_t orn_gemm_multi(orn_ctx* ctx, const orn_linear* const* lins, int32_t n, c
   int ld[4];
   for (int j = 0; j < n; ++j) {
     if (!lins[j] || !ys[j]) return ORN_ERR_ARG;
+    if (lins[j]->K % 64) ORN_FAIL(ctx, ORN_ERR_ARG, "gemm: K must be a multiple of 64");
     ld[j] = lins[j]->O;
   }
   return f_qgemm_multi(ctx, ctx->stream, lins, ys, ld, n, x, M, nullptr, nullptr, out_f32, 0);

@@ -579,6 +579,7 @@ int32_t orn_batch_destroy(orn_batch* bt) {
 int32_t orn_batch_create(orn_model* m, int32_t B, int32_t T_max, int32_t cap, int32_t flags, orn_batch** out) {
   if (!m || !out) return ORN_ERR_ARG;
   *out = nullptr;
+  if (m->dec != nullptr) ORN_FAIL(m->ctx, ORN_ERR_ARG, "batch_create: the batched engine runs the Qwen3.5-MoE trunk only");
   CK(orn_model_finalize(m));
   orn_ctx* ctx = m->ctx;
   const orn_config& c = m->cfg;

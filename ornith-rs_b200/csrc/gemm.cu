@@ -42,6 +42,7 @@
 #include <string>
 #include <utility>
 
+#include "act.cuh"
 #include "fused.h"
 #include "orn_internal.h"
 #include "orn_quant.cuh"
@@ -71,6 +72,8 @@ struct GemmJob {
   int ldy;             // elements between output rows
   bf16_t* y;
   float* y_f32;        // non-null: float32 output instead of bfloat16
+  const bf16_t* bias;  // bf16 weights only, nullable: added to the product, then the activation
+  ActParams act;
 };
 struct GemmParams {
   int njobs;
@@ -79,7 +82,7 @@ struct GemmParams {
   const int* n_items;  // grouped: device count
   int dense_items;     // dense: feature tiles x token groups
   int rows;            // rows of x (dense) / of the sorted row space (grouped)
-  int K;
+  int K, KB;           // row length, K blocks of 64 (bf16 rows may end inside the last one: TMA fills zeros)
   const uint32_t* row_map;   // nullable: output row of sorted row p
   int BN, NT, stages /*IN ring*/, w_stages /*W ring*/, f_tiles;
   uint32_t stage_bytes;
@@ -377,7 +380,7 @@ ORN_D bool get_item(const GemmParams& P, int w, int n_items, Item& it) {
   if (P.items != nullptr) {
     const int4 v = P.items[w];
     it.e = v.x; it.tok0 = v.y; it.ntok = v.z; it.ft = v.w;
-    it.kb0 = 0; it.kb1 = P.K / BK; it.tile = w; it.split = 0; it.job = 0;
+    it.kb0 = 0; it.kb1 = P.KB; it.tile = w; it.split = 0; it.job = 0;
     while (it.job + 1 < P.njobs && it.ft >= P.job[it.job + 1].tile0) ++it.job;
     it.ft -= P.job[it.job].tile0;
   } else {
@@ -390,7 +393,7 @@ ORN_D bool get_item(const GemmParams& P, int w, int n_items, Item& it) {
     it.ft -= P.job[it.job].tile0;
     it.tok0 = g * P.NT * P.BN;
     it.ntok = min(P.NT * P.BN, P.rows - it.tok0);
-    const int KB = P.K / BK, per = (KB + P.splits - 1) / P.splits;
+    const int KB = P.KB, per = (KB + P.splits - 1) / P.splits;
     it.tile = tile; it.split = w - tile * P.splits;
     it.kb0 = it.split * per; it.kb1 = min(KB, it.kb0 + per);
   }
@@ -576,6 +579,11 @@ __global__ void __launch_bounds__(gemm_threads(DQW), DQW == 4 ? 4 : 1) k_qgemm(c
       const GemmJob& J = P.job[w.job];
       const int fo = w.ft * BM + q * 32 + lane;  // TMEM lane = feature
       const int nt = (w.ntok + P.BN - 1) / P.BN;
+      float ep_bias = 0.f, ep_a = 0.f, ep_b = 0.f;
+      if (kDirect) {
+        act_prepare(J.act, ep_a, ep_b);
+        if (J.bias != nullptr && fo < J.O) ep_bias = bf2f(J.bias[fo]);
+      }
       // split-K items store f32 partials [token][128 features] instead of results
       float* part = P.splits > 1 ? P.partial + (size_t)(w.tile * P.splits + w.split) * (size_t)(P.NT * P.BN) * BM : nullptr;
       for (int t = 0; t < nt; ++t) {
@@ -596,8 +604,10 @@ __global__ void __launch_bounds__(gemm_threads(DQW), DQW == 4 ? 4 : 1) k_qgemm(c
               const int tok = t * P.BN + c0 + j;
               if (tok < w.ntok) {
                 const size_t orow = P.row_map != nullptr ? P.row_map[w.tok0 + tok] : (size_t)(w.tok0 + tok);
-                if (J.y_f32 != nullptr) J.y_f32[orow * J.ldy + fo] = __uint_as_float(v[j]);
-                else J.y[orow * J.ldy + fo] = f2bf(__uint_as_float(v[j]));
+                float r = __uint_as_float(v[j]);
+                if (kDirect) r = act_apply(J.act.kind, r + ep_bias, ep_a, ep_b);
+                if (J.y_f32 != nullptr) J.y_f32[orow * J.ldy + fo] = r;
+                else J.y[orow * J.ldy + fo] = f2bf(r);
               }
             }
           }
@@ -644,8 +654,10 @@ __global__ void __launch_bounds__(gemm_threads(DQW), DQW == 4 ? 4 : 1) k_qgemm(c
 #pragma unroll
               for (int e = 0; e < 4; ++e)
                 if (feat + e < J.O) {
-                  if (J.y_f32 != nullptr) J.y_f32[orow * J.ldy + feat + e] = r4[e];
-                  else J.y[orow * J.ldy + feat + e] = f2bf(r4[e]);
+                  float r = r4[e];
+                  if (kDirect) r = act_apply(J.act.kind, r + (J.bias != nullptr ? bf2f(J.bias[feat + e]) : 0.f), ep_a, ep_b);
+                  if (J.y_f32 != nullptr) J.y_f32[orow * J.ldy + feat + e] = r;
+                  else J.y[orow * J.ldy + feat + e] = f2bf(r);
                 }
             }
           }
@@ -810,14 +822,18 @@ int f_qgemm(orn_ctx* ctx, cudaStream_t s, const orn_linear* L, const bf16_t* x, 
 // Up to four matrices of one format and row length over the same rows in ONE launch (the projections
 // of a layer that share their input): their feature tiles form one tile space.  n == 1 is f_qgemm.
 int f_qgemm_multi(orn_ctx* ctx, cudaStream_t s, const orn_linear* const* Ls, void* const* ys, const int* ldys, int n,
-                  const bf16_t* x, int rows, const QGemmGroup* grp, void* scratch, int out_f32, int bn_force) {
+                  const bf16_t* x, int rows, const QGemmGroup* grp, void* scratch, int out_f32, int bn_force,
+                  const QGemmEpi* epi, int ldx) {
   if (rows < 1) return ORN_OK;
   if (n < 1 || n > kMaxJobs) ORN_FAIL(ctx, ORN_ERR_ARG, "gemm: 1..4 matrices per launch");
   const orn_linear* L = Ls[0];
   for (int j = 1; j < n; ++j)
     if (Ls[j]->kind != L->kind || Ls[j]->K != L->K || Ls[j]->E != L->E)
       ORN_FAIL(ctx, ORN_ERR_ARG, "gemm: the matrices of one launch share format and row length");
-  if (L->K % BK) ORN_FAIL(ctx, ORN_ERR_ARG, "gemm: K must be a multiple of 64");
+  if (L->K % (L->kind == ORN_BF16 ? 8 : BK)) ORN_FAIL(ctx, ORN_ERR_ARG, "gemm: K must be a multiple of 64 (bf16 rows: of 8)");
+  if (epi != nullptr && L->kind != ORN_BF16) ORN_FAIL(ctx, ORN_ERR_ARG, "gemm: bias and activation go with bf16 weights");
+  if (ldx <= 0) ldx = L->K;
+  if (ldx % 8 || ldx < L->K) ORN_FAIL(ctx, ORN_ERR_ARG, "gemm: the row stride of x must be a multiple of 8 and hold a row");
   if ((reinterpret_cast<uintptr_t>(x) & 15) != 0) ORN_FAIL(ctx, ORN_ERR_ARG, "gemm: x must be 16-byte aligned");
   if (grp == nullptr && L->E != 1) ORN_FAIL(ctx, ORN_ERR_ARG, "gemm: a routed weight goes through the grouped form");
   EncodeTiledFn enc = encode_tiled();
@@ -828,11 +844,14 @@ int f_qgemm_multi(orn_ctx* ctx, cudaStream_t s, const orn_linear* const* Ls, voi
   for (int j = 0; j < n; ++j) {
     GemmJob& J = P.job[j];
     J.O = Ls[j]->O; J.tile0 = P.f_tiles; J.ldy = ldys[j];
-    J.y = out_f32 ? nullptr : reinterpret_cast<bf16_t*>(ys[j]);
-    J.y_f32 = out_f32 ? reinterpret_cast<float*>(ys[j]) : nullptr;
+    const bool f32 = epi != nullptr ? epi[j].out_f32 : out_f32 != 0;
+    J.y = f32 ? nullptr : reinterpret_cast<bf16_t*>(ys[j]);
+    J.y_f32 = f32 ? reinterpret_cast<float*>(ys[j]) : nullptr;
+    J.bias = epi != nullptr ? epi[j].bias : nullptr;
+    J.act = epi != nullptr ? epi[j].act : ActParams();
     P.f_tiles += (Ls[j]->O + BM - 1) / BM;
   }
-  P.K = L->K; P.rows = rows; P.err = ctx->dev_err;
+  P.K = L->K; P.KB = (L->K + BK - 1) / BK; P.rows = rows; P.err = ctx->dev_err;
   P.row_map = grp ? grp->row_map : nullptr;
   // token-tile width: wide tiles when there are many tokens per weight tile, narrow ones otherwise
   int per = grp ? (rows + L->E - 1) / L->E : rows;  // expected tokens per weight tile
@@ -865,14 +884,14 @@ int f_qgemm_multi(orn_ctx* ctx, cudaStream_t s, const orn_linear* const* Ls, voi
   // (O, K) only, never on the row count, so that a row's bits do not depend on how many rows share
   // the launch.
   P.splits = 1; P.partial = nullptr; P.arrivals = nullptr;
-  if (grp == nullptr && rows <= kSplitMaxRows && L->K / BK >= 8) {
+  if (grp == nullptr && rows <= kSplitMaxRows && P.KB >= 8) {
     const int tiles = P.f_tiles * ((rows + P.NT * BN - 1) / (P.NT * BN));
     // one round of items over the SMs, two CTAs on each where the tiles alone would leave SMs idle
     // (97 tiles of an input projection: three splits instead of none)
     int sp = std::max(1, (tiles > ctx->sm_count / 2 ? 2 * ctx->sm_count : ctx->sm_count) / tiles);
-    sp = std::min(sp, std::min(8, L->K / BK / 4));               // at least 4 K blocks per item
+    sp = std::min(sp, std::min(8, P.KB / 4));               // at least 4 K blocks per item
     if (sp > 1) {                                                 // no split may be empty
-      const int KBn = L->K / BK, per = (KBn + sp - 1) / sp;
+      const int KBn = P.KB, per = (KBn + sp - 1) / sp;
       sp = (KBn + per - 1) / per;
     }
     const int groups = (rows + P.NT * BN - 1) / (P.NT * BN);
@@ -945,7 +964,7 @@ int f_qgemm_multi(orn_ctx* ctx, cudaStream_t s, const orn_linear* const* Ls, voi
                CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
   };
   bool ok = encode(&maps.x, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, const_cast<bf16_t*>(x), (uint64_t)L->K, (uint64_t)rows,
-                   (uint64_t)L->K * 2, BK, (uint32_t)BN, CU_TENSOR_MAP_SWIZZLE_128B);
+                   (uint64_t)ldx * 2, BK, (uint32_t)BN, CU_TENSOR_MAP_SWIZZLE_128B);
   for (int j = 0; j < n; ++j) {
     const orn_linear* Lj = Ls[j];
     WeightMaps& wm = maps.w[j];

@@ -14,6 +14,8 @@
 #include <memory>
 #include <type_traits>
 
+#include "arch.h"
+#include "dense.h"
 #include "fused.h"
 #include "model_types.h"
 #include "orn_internal.h"
@@ -23,6 +25,8 @@
     int rc__ = (call);               \
     if (rc__ != ORN_OK) return rc__; \
   } while (0)
+
+extern const orn_arch kArchQwen35;
 
 namespace {
 
@@ -158,7 +162,7 @@ int load_moe(orn_model* m, const std::string& p, Moe& moe) {
 
 // resolve every name the forward pass needs (TextModel::load, qwen3_5.rs:102-158;
 // MtpHead::load, mtp.rs:96-143)
-int finalize(orn_model* m) {
+int qwen_finalize(orn_model* m) {
   if (m->finalized) return ORN_OK;
   const orn_config& c = m->cfg;
   const int H = c.hidden, D = conv_dim(c), VD = c.gdn_v_heads * c.gdn_head_dim;
@@ -232,6 +236,8 @@ int finalize(orn_model* m) {
   m->finalized = true;
   return ORN_OK;
 }
+
+int finalize(orn_model* m) { return m->arch->finalize(m); }
 
 // ------------------------------------------------------------------ blocks
 // sparse_moe_block (src/ops/moe.rs:662-741); with bf16 weights it is
@@ -496,20 +502,29 @@ int trunk_finish(orn_model* m, orn_cache* cc, int T, bool capture, bf16_t* norme
 }
 
 // the trunk over T <= kMaxRows rows whose ids are already on the device
-int forward_dev(orn_model* m, orn_cache* cc, const uint32_t* dev_ids, int T, bool capture,
-                bf16_t* normed_out, bf16_t* pre_norm_out) {
+int qwen_forward(orn_model* m, orn_cache* cc, const uint32_t* dev_ids, int T, bool capture, void* normed_v, void* pre_norm_v) {
+  bf16_t *normed_out = (bf16_t*)normed_v, *pre_norm_out = (bf16_t*)pre_norm_v;
   CK(trunk_layers(m, cc, dev_ids, T, capture));
   return trunk_finish(m, cc, T, capture, normed_out, pre_norm_out, nullptr, nullptr);
 }
 
 // trunk + lm_head + greedy for every row: tokens land in dev_tokens, the
 // post-norm hidden rows in normed_out
-int forward_greedy_dev(orn_model* m, orn_cache* cc, const uint32_t* dev_ids, int T, bool capture,
-                       bf16_t* normed_out, uint32_t* dev_tokens) {
+int qwen_forward_greedy(orn_model* m, orn_cache* cc, const uint32_t* dev_ids, int T, bool capture, void* normed_v,
+                        uint32_t* dev_tokens) {
+  bf16_t* normed_out = (bf16_t*)normed_v;
   Workspace& w = m->ws;
   CK(trunk_layers(m, cc, dev_ids, T, capture));
   CK(trunk_finish(m, cc, T, capture, normed_out, nullptr, m->lm_head, w.logits));
   return k_greedy(m->ctx, m->ctx->stream, w.logits, T, m->lm_head->O, 1, dev_tokens, w.greedy_scratch);
+}
+
+int forward_dev(orn_model* m, orn_cache* cc, const uint32_t* dev_ids, int T, bool capture, void* normed_out, void* pre_norm_out) {
+  return m->arch->forward(m, cc, dev_ids, T, capture, normed_out, pre_norm_out);
+}
+int forward_greedy_dev(orn_model* m, orn_cache* cc, const uint32_t* dev_ids, int T, bool capture, void* normed_out,
+                       uint32_t* dev_tokens) {
+  return m->arch->forward_greedy(m, cc, dev_ids, T, capture, normed_out, dev_tokens);
 }
 
 int upload_ids(orn_model* m, const uint32_t* host_ids, int T) {
@@ -656,7 +671,7 @@ int run_step(orn_model* m, orn_cache* c, int kind /*0 cycle, 1 ar, 2 prefill row
   if (kind == 0 && c->h_mtp_pos + want > m->cfg.max_ctx) ORN_FAIL(ctx, ORN_ERR_STATE, "mtp: context exceeds max_ctx");
   static int no_graph = -1;
   if (no_graph < 0) { const char* e = getenv("ORN_NO_GRAPH"); no_graph = (e && e[0] == '1') ? 1 : 0; }
-  const bool eager = no_graph || ctx->kt != nullptr;  // per-kernel times need eager launches
+  const bool eager = no_graph || ctx->kt != nullptr || m->tap != nullptr;  // per-kernel times and taps need eager launches
   if (g.exec != nullptr && use_frspec && g.fr_gen != m->fr_gen) {
     // the pruned head was replaced since this graph was captured: its kernel arguments point at
     // freed memory.  Drop it; the shape is run eagerly once and captured again.
@@ -677,7 +692,7 @@ int run_step(orn_model* m, orn_cache* c, int kind /*0 cycle, 1 ar, 2 prefill row
     if (kind == 1) return ar_body(m, c);
     return forward_dev(m, c, m->ws.ids, n_rows, false, nullptr, nullptr);  // a window of prompt rows
   };
-  if (g.seen == 0 || eager || !use_fused(m) || g.exec != nullptr) {
+  if (g.seen == 0 || eager || !m->arch->graphs(m) || g.exec != nullptr) {
     g.seen += 1;
     return body();
   }
@@ -905,33 +920,46 @@ int prefill_wide(orn_model* m, orn_cache* cc, int T, bf16_t* normed_out /*nullab
   return ORN_OK;
 }
 
+bool qwen_chunked(const orn_model*) { return use_wide_prefill() && use_fused_env(); }
+int qwen_chunk(orn_model* m, orn_cache* cc, const uint32_t* host_ids, int T, void* normed_out) {
+  CK(wide_reserve(m, T));
+  ORN_CHECK_CUDA(m->ctx, cudaMemcpyAsync(m->wide.ids, host_ids, sizeof(uint32_t) * (size_t)T, cudaMemcpyHostToDevice, m->ctx->stream));
+  return prefill_wide(m, cc, T, (bf16_t*)normed_out);
+}
+int qwen_logits(orn_model* m, const void* rows, int T, float* dev_out) {
+  if (T <= kMaxRows) return k_gemv(m->ctx, m->ctx->stream, m->lm_head, (const bf16_t*)rows, T, dev_out, 1);
+  return f_qgemm(m->ctx, m->ctx->stream, m->lm_head, (const bf16_t*)rows, T, dev_out, m->lm_head->O, nullptr, nullptr, 1);
+}
+int qwen_head_greedy(orn_model* m, const void* rows, int T, uint32_t* dev_tokens, void* dev_logits) {
+  return head_greedy_dev(m, m->lm_head, (const bf16_t*)rows, T, 1, dev_logits ? (bf16_t*)dev_logits : m->ws.logits, dev_tokens);
+}
+
+size_t row_bytes(const orn_model* m) { return (size_t)m->row_ld * (m->dtype == ORN_DT_F32 ? 4 : 2); }
+
 // generate::prefill (src/generate.rs:90-136): everything but the last prompt
 // token.  Rows are computed with one-row arithmetic, so the chunk width (the
 // reference's prefill_step) cannot change the result; chunks are cut to the
 // widest window a forward call takes.
 int prefill(orn_model* m, orn_cache* cc, const uint32_t* prompt, int n, int prefill_step, int* done_out,
-            bf16_t* normed_out = nullptr, int keep_last = 1) {
+            void* normed_out = nullptr, int keep_last = 1) {
+  const orn_arch* arch = m->arch;
   int done = 0;
   int step = prefill_step < 1 ? 1 : prefill_step;
+  auto row = [&](int i) -> void* { return normed_out ? (uint8_t*)normed_out + (size_t)i * row_bytes(m) : nullptr; };
   while (n - done > keep_last) {
     int chunk = std::min(step, n - done - keep_last);
     int off = 0;
-    if (chunk >= kWideMinRows && use_wide_prefill() && use_fused_env()) {
+    if (chunk >= arch->chunk_min && arch->chunked(m)) {
       // a chunk wide enough for the tensor cores (the reference's tile path, kquant.rs:783-812)
-      chunk = std::min(chunk, kWideMaxRows);
-      CK(wide_reserve(m, chunk));
-      ORN_CHECK_CUDA(m->ctx, cudaMemcpyAsync(m->wide.ids, prompt + done, sizeof(uint32_t) * (size_t)chunk,
-                                             cudaMemcpyHostToDevice, m->ctx->stream));
-      CK(prefill_wide(m, cc, chunk, normed_out ? normed_out + (size_t)done * m->cfg.hidden : nullptr));
+      chunk = std::min(chunk, arch->chunk_max);
+      CK(arch->chunk(m, cc, prompt + done, chunk, row(done)));
       off = chunk;
     }
     while (off < chunk) {
       int t = std::min(kMaxRows, chunk - off);
       CK(upload_ids(m, prompt + done + off, t));
-      if (normed_out != nullptr)
-        CK(forward_dev(m, cc, m->ws.ids, t, false, normed_out + (size_t)(done + off) * m->cfg.hidden, nullptr));
-      else
-        CK(run_step(m, cc, 2, t - 1, false));  // the same rows as forward_dev, replayed as a graph
+      if (normed_out != nullptr) CK(forward_dev(m, cc, m->ws.ids, t, false, row(done + off), nullptr));
+      else CK(run_step(m, cc, 2, t - 1, false));  // the same rows as forward_dev, replayed as a graph
       off += t;
     }
     CK(orn_sync(m->ctx));  // the reference drains the queue after each chunk (generate.rs:128-131)
@@ -951,6 +979,7 @@ uint64_t splitmix64(uint64_t x) {
 }  // namespace
 
 int orn_model_finalize(orn_model* m) { return finalize(m); }
+int orn_cache_commit(orn_cache* c, int keep, int ring_step) { return commit(c, keep, ring_step); }
 bool orn_wide_exact() { return wide_exact(); }
 int orn_conv_dim(const orn_config& c) { return conv_dim(c); }
 
@@ -967,6 +996,8 @@ int32_t orn_model_create(orn_ctx* ctx, const orn_config* cfg, orn_model** out) {
     ORN_FAIL(ctx, ORN_ERR_ARG, "model_create: unsupported dimensions");
   orn_model* m = new orn_model();
   m->ctx = ctx;
+  m->arch = &kArchQwen35;
+  m->row_ld = cfg->hidden;
   m->cfg = *cfg;
   *out = m;
   return ORN_OK;
@@ -983,6 +1014,8 @@ int32_t orn_model_destroy(orn_model* m) {
   cudaFree(m->fr_ids);
   for (int i = 0; i < 4; ++i)
     if (m->ev[i]) cudaEventDestroy(m->ev[i]);
+  if (m->arch && m->arch->release) m->arch->release(m);
+  cudaFree(m->step_rows); cudaFree(m->step_sel); cudaFree(m->step_idx);
   delete m;
   return ORN_OK;
 }
@@ -1045,9 +1078,7 @@ size_t orn_model_weight_bytes(const orn_model* m) {
 // Random-init in the mix the benchmark names: expert gate/up Q4_K, expert down
 // Q6_K (shared expert: the same formats), every other matrix 8-bit affine, the
 // small gated-delta projections and the whole MTP head bf16.
-int32_t orn_model_init_random(orn_model* m, uint64_t seed) {
-  if (!m) return ORN_ERR_ARG;
-  if (m->finalized) ORN_FAIL(m->ctx, ORN_ERR_STATE, "model_init_random: model already in use");
+static int qwen_init_random(orn_model* m, uint64_t seed) {
   orn_ctx* ctx = m->ctx;
   const orn_config& c = m->cfg;
   const int H = c.hidden, D = conv_dim(c), VD = c.gdn_v_heads * c.gdn_head_dim;
@@ -1128,6 +1159,12 @@ int32_t orn_model_init_random(orn_model* m, uint64_t seed) {
   return orn_sync(ctx);
 }
 
+int32_t orn_model_init_random(orn_model* m, uint64_t seed) {
+  if (!m) return ORN_ERR_ARG;
+  if (m->finalized) ORN_FAIL(m->ctx, ORN_ERR_STATE, "model_init_random: model already in use");
+  return m->arch->init_random(m, seed);
+}
+
 int32_t orn_frspec_set(orn_model* m, const uint32_t* host_ids, int32_t n) {
   if (!m || !host_ids || n < 1) return ORN_ERR_ARG;
   CK(finalize(m));
@@ -1166,13 +1203,9 @@ int32_t orn_frspec_load(orn_model* m, const char* ids_path) {
 }
 
 // ------------------------------------------------------------------ caches
-int32_t orn_cache_create(orn_model* m, orn_cache** out) {
-  if (!m || !out) return ORN_ERR_ARG;
-  *out = nullptr;
-  CK(finalize(m));
+static int qwen_cache_init(orn_cache* k) {
+  orn_model* m = k->m;
   const orn_config& c = m->cfg;
-  orn_cache* k = new orn_cache();
-  k->m = m;
   k->kc.assign(c.n_layers, nullptr); k->vc.assign(c.n_layers, nullptr);
   k->conv.assign(c.n_layers, nullptr); k->ring.assign(c.n_layers, nullptr);
   const size_t kvsz = sizeof(bf16_t) * (size_t)c.n_kv_heads * c.max_ctx * c.head_dim;
@@ -1192,12 +1225,22 @@ int32_t orn_cache_create(orn_model* m, orn_cache** out) {
   }
   if (rc == ORN_OK) rc = orn_alloc(m->ctx, kvsz, (void**)&k->mtp_kc);
   if (rc == ORN_OK) rc = orn_alloc(m->ctx, kvsz, (void**)&k->mtp_vc);
-  if (rc == ORN_OK) rc = orn_alloc(m->ctx, 3 * sizeof(int), (void**)&k->pos);
   k->n_gdn = (int)table.size();
   if (rc == ORN_OK && k->n_gdn) {
     rc = orn_alloc(m->ctx, sizeof(bf16_t*) * table.size(), (void**)&k->conv_table);
     if (rc == ORN_OK) rc = orn_upload(m->ctx, k->conv_table, table.data(), sizeof(bf16_t*) * table.size());
   }
+  return rc;
+}
+
+int32_t orn_cache_create(orn_model* m, orn_cache** out) {
+  if (!m || !out) return ORN_ERR_ARG;
+  *out = nullptr;
+  CK(finalize(m));
+  orn_cache* k = new orn_cache();
+  k->m = m;
+  int rc = orn_alloc(m->ctx, 3 * sizeof(int), (void**)&k->pos);
+  if (rc == ORN_OK) rc = m->arch->cache_init(k);
   if (rc != ORN_OK) { orn_cache_destroy(k); return rc; }
   if (cudaMallocHost((void**)&k->mailbox_h, 16 * sizeof(uint32_t)) != cudaSuccess) {
     orn_cache_destroy(k);
@@ -1220,13 +1263,13 @@ int32_t orn_cache_destroy(orn_cache* k) {
   for (auto& g : k->graphs)
     if (g.second.exec) cudaGraphExecDestroy(g.second.exec);
   if (k->mailbox_h) cudaFreeHost(k->mailbox_h);
+  if (k->m->arch->cache_release) k->m->arch->cache_release(k);
   delete k;
   return ORN_OK;
 }
 
 // make_cache (cache.rs:160-181): zero conv windows and states, empty KV
-int32_t orn_cache_reset(orn_cache* k) {
-  if (!k) return ORN_ERR_ARG;
+static int qwen_cache_reset(orn_cache* k) {
   orn_model* m = k->m;
   const orn_config& c = m->cfg;
   const size_t ssz = sizeof(float) * (size_t)c.gdn_v_heads * 128 * 128;
@@ -1236,6 +1279,12 @@ int32_t orn_cache_reset(orn_cache* k) {
       CK(orn_memset(m->ctx, k->conv[i], 0, csz));
       CK(orn_memset(m->ctx, k->ring[i], 0, ssz * kRing));
     }
+  return ORN_OK;
+}
+int32_t orn_cache_reset(orn_cache* k) {
+  if (!k) return ORN_ERR_ARG;
+  orn_model* m = k->m;
+  CK(m->arch->cache_reset(k));
   CK(orn_memset(m->ctx, k->pos, 0, 3 * sizeof(int)));
   k->h_pos = k->h_cur = k->h_mtp_pos = 0;
   k->cap_T = 0;
@@ -1271,6 +1320,57 @@ int32_t orn_prefill(orn_model* m, orn_cache* c, const uint32_t* host_ids, int32_
   return orn_sync(m->ctx);
 }
 
+int32_t orn_step(orn_model* m, orn_cache* c, const uint32_t* host_ids, int32_t n, int32_t prefill_step, const int32_t* host_want,
+                 int32_t n_want, float* dev_logits) {
+  if (!m || !c || !host_ids || n < 1 || n_want < 0 || (n_want > 0 && (!host_want || !dev_logits))) return ORN_ERR_ARG;
+  orn_ctx* ctx = m->ctx;
+  CK(finalize(m));
+  for (int i = 0; i < n_want; ++i)
+    if (host_want[i] < 0 || host_want[i] >= n || (i && host_want[i] <= host_want[i - 1]))
+      ORN_FAIL(ctx, ORN_ERR_ARG, "step: wanted places must ascend within the tokens");
+  for (int i = 0; i < n; ++i)
+    if (host_ids[i] >= (uint32_t)m->cfg.vocab) ORN_FAIL(ctx, ORN_ERR_ARG, "step: token id outside the vocabulary");
+  const int piece = std::min(n, std::max(1, std::min(prefill_step, m->arch->chunk_max)));
+  if (m->step_cap < piece) {
+    ORN_CHECK_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+    cudaFree(m->step_rows); cudaFree(m->step_sel); cudaFree(m->step_idx);
+    m->step_rows = m->step_sel = nullptr; m->step_idx = nullptr; m->step_cap = 0;
+    CK(orn_alloc(ctx, (size_t)piece * row_bytes(m), &m->step_rows));
+    CK(orn_alloc(ctx, (size_t)piece * row_bytes(m), &m->step_sel));
+    CK(orn_alloc(ctx, (size_t)piece * sizeof(int), (void**)&m->step_idx));
+    m->step_cap = piece;
+  }
+  m->tap_rows = n;
+  int at = 0, w0 = 0;
+  while (at < n) {
+    const int t = std::min(piece, n - at);
+    int w1 = w0;
+    std::vector<int> idx;
+    while (w1 < n_want && host_want[w1] < at + t) idx.push_back(host_want[w1++] - at);
+    m->tap_at = at;
+    int done = 0;
+    const int pos0 = c->h_pos;
+    CK(prefill(m, c, host_ids + at, t, t, &done, idx.empty() ? nullptr : m->step_rows, 0));
+    if (c->h_pos != pos0 + t) ORN_FAIL(ctx, ORN_ERR_STATE, "step: the cache did not advance by the tokens");
+    if (!idx.empty()) {
+      CK(orn_upload(ctx, m->step_idx, idx.data(), idx.size() * sizeof(int)));
+      CK(k_gather_act_rows(ctx, ctx->stream, m->step_rows, m->step_idx, (int)idx.size(), m->row_ld, m->step_sel, m->dtype == ORN_DT_F32));
+      CK(m->arch->logits(m, m->step_sel, (int)idx.size(), dev_logits + (size_t)w0 * m->cfg.vocab));
+      CK(orn_sync(ctx));
+    }
+    w0 = w1;
+    at += t;
+  }
+  return ORN_OK;
+}
+
+int32_t orn_model_tap(orn_model* m, float* dev_tap) {
+  if (!m) return ORN_ERR_ARG;
+  if (dev_tap && m->dec == nullptr) ORN_FAIL(m->ctx, ORN_ERR_ARG, "tap: this architecture has none");
+  m->tap = dev_tap;
+  return ORN_OK;
+}
+
 int32_t orn_cache_rewind(orn_cache* c, int32_t keep) {
   if (!c) return ORN_ERR_ARG;
   if (c->cap_T == 0) ORN_FAIL(c->m->ctx, ORN_ERR_STATE, "cache_rewind: no captured window");
@@ -1284,8 +1384,7 @@ int32_t orn_head_greedy(orn_model* m, const uint16_t* dev_hidden, int32_t T, uin
   if (!m || !dev_hidden || !host_tokens) return ORN_ERR_ARG;
   CK(finalize(m));
   if (T < 1 || T > kMaxRows) ORN_FAIL(m->ctx, ORN_ERR_ARG, "head_greedy: 1..4 rows per call");
-  bf16_t* logits = dev_logits_out ? dev_logits_out : m->ws.logits;
-  CK(head_greedy_dev(m, m->lm_head, dev_hidden, T, 1, logits, m->ws.targets));
+  CK(m->arch->head_greedy(m, dev_hidden, T, m->ws.targets, dev_logits_out));
   return orn_download(m->ctx, host_tokens, m->ws.targets, sizeof(uint32_t) * (size_t)T);
 }
 
@@ -1535,3 +1634,23 @@ int32_t orn_moe_block(orn_ctx* ctx, const orn_linear* gate, const orn_linear* sw
 }
 
 }  // extern "C"
+
+// ------------------------------------------------------------------ the model registry
+static bool qwen_graphs(const orn_model* m) { return use_fused(m); }
+
+extern const orn_arch kArchQwen35 = {
+    "qwen3_5_moe",   qwen35_load,     nullptr,      qwen_finalize,       qwen_init_random, nullptr,
+    qwen_cache_init, qwen_cache_reset, nullptr,     qwen_forward,        qwen_forward_greedy,
+    kWideMinRows,    kWideMaxRows,    qwen_chunked, qwen_chunk,          qwen_logits,      qwen_head_greedy,
+    qwen_graphs,
+};
+
+// The "architecture" of a config.json names its entry; the reference's own files have none and mean Qwen3.5-MoE.
+const orn_arch* orn_arch_of_config(const orna::JVal& cfg) {
+  static const orn_arch* const all[] = {&kArchQwen35, &kArchPeratar};
+  const orna::JVal* a = cfg.get("architecture");
+  if (a == nullptr || a->type != orna::JVal::Str) return &kArchQwen35;
+  for (const orn_arch* e : all)
+    if (a->str == e->name) return e;
+  return nullptr;
+}

@@ -76,8 +76,20 @@ struct WideWs {
 
 using namespace ornm;
 
+struct orn_arch;     // arch.h
+struct orn_decoder;  // decoder.cu
+
 struct orn_model {
   orn_ctx* ctx = nullptr;
+  const orn_arch* arch = nullptr;   // the registry entry that runs this model
+  orn_decoder* dec = nullptr;       // its own state (decoder.cu)
+  int dtype = ORN_DT_BF16;          // activation type
+  int row_ld = 0;                   // elements per hidden row in the API's row buffers
+  float* tap = nullptr;             // orn_model_tap: the stream after every layer
+  int tap_rows = 0, tap_at = 0;     // rows per layer in the tap of the running call, first row of the running pass
+  void *step_rows = nullptr, *step_sel = nullptr;  // orn_step: rows after the final norm, the wanted ones
+  int* step_idx = nullptr;
+  int step_cap = 0;
   orn_config cfg{};
   std::map<std::string, orn_linear*> lins;
   std::map<std::string, Tensor> tensors;
@@ -101,6 +113,7 @@ struct orn_model {
 
 struct orn_cache {
   orn_model* m = nullptr;
+  std::vector<void*> latent;         // per layer (latent attention): [max_ctx][row], shared by layers that read another's
   std::vector<bf16_t*> kc, vc;       // per layer (attention layers)
   std::vector<bf16_t*> conv;         // per layer (gdn): [S + kMaxRows, D]
   std::vector<float*> ring;          // per layer (gdn): [kRing][Hv,128,128]
@@ -124,6 +137,8 @@ struct orn_cache {
 
 // resolves every weight name the forward pass needs and builds the scratch (idempotent)
 int orn_model_finalize(orn_model* m);
+// `keep` rows of the last pass stand: positions advance (and, where a model has them, conv windows and states)
+int orn_cache_commit(orn_cache* c, int keep, int ring_step);
 // ORN_WIDE_EXACT=1: wide paths compute their products with the row-invariant mat-vec kernels
 bool orn_wide_exact();
 int orn_conv_dim(const orn_config& c);

@@ -263,4 +263,5 @@ int k_sdpa_decode(orn_ctx* ctx, cudaStream_t s, const bf16_t* q, const bf16_t* k
 // sample.cu
 int k_greedy(orn_ctx* ctx, cudaStream_t s, const bf16_t* logits, int T, int V, int normalize,
              uint32_t* tokens, float* scratch /* [T, 2*ceil(V/1024)] */);
+int k_greedy_f32(orn_ctx* ctx, cudaStream_t s, const float* logits, int T, int V, uint32_t* tokens, float* scratch);
 size_t greedy_scratch_floats(int T, int V);

@@ -16,11 +16,15 @@
 
 namespace {
 
+ORN_D float logit_of(bf16_t v) { return bf2f(v); }
+ORN_D float logit_of(float v) { return v; }
+
+template <typename TL>
 __global__ void __launch_bounds__(256)
-lse_chunk_kernel(const bf16_t* __restrict__ logits, int V, int nc, float* __restrict__ scratch) {
+lse_chunk_kernel(const TL* __restrict__ logits, int V, int nc, float* __restrict__ scratch) {
   __shared__ float red[32];
   const int b = blockIdx.x, t = blockIdx.y;
-  const bf16_t* x = logits + (int64_t)t * V + (int64_t)b * 1024;
+  const TL* x = logits + (int64_t)t * V + (int64_t)b * 1024;
   const int n = min(1024, V - b * 1024);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   float v[4];
@@ -28,7 +32,7 @@ lse_chunk_kernel(const bf16_t* __restrict__ logits, int V, int nc, float* __rest
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     int idx = 4 * threadIdx.x + i;
-    v[i] = idx < n ? bf2f(x[idx]) : -INFINITY;
+    v[i] = idx < n ? logit_of(x[idx]) : -INFINITY;
     m = fmaxf(m, v[i]);
   }
   m = warp_max(m);
@@ -54,8 +58,9 @@ lse_chunk_kernel(const bf16_t* __restrict__ logits, int V, int nc, float* __rest
   }
 }
 
+template <typename TL>
 __global__ void __launch_bounds__(256)
-greedy_finish_kernel(const bf16_t* __restrict__ logits, int V, int nc, int normalize,
+greedy_finish_kernel(const TL* __restrict__ logits, int V, int nc, int normalize,
                      const float* __restrict__ scratch, uint32_t* __restrict__ tokens) {
   extern __shared__ float sh[];  // m[nc], e[nc]
   __shared__ float red[32];
@@ -95,14 +100,14 @@ greedy_finish_kernel(const bf16_t* __restrict__ logits, int V, int nc, int norma
   }
   __syncthreads();
   const int b = s_chunk;
-  const bf16_t* x = logits + (int64_t)t * V + (int64_t)b * 1024;
+  const TL* x = logits + (int64_t)t * V + (int64_t)b * 1024;
   const int n = min(1024, V - b * 1024);
   unsigned int best = 0xffffffffu;
 #pragma unroll
   for (int i = 3; i >= 0; --i) {
     int idx = 4 * threadIdx.x + i;
     if (idx < n) {
-      float lp = normalize ? bfr(bf2f(x[idx]) - s_lse) : bf2f(x[idx]);
+      float lp = normalize ? bfr(logit_of(x[idx]) - s_lse) : logit_of(x[idx]);
       if (lp == s_target) best = (unsigned int)(b * 1024 + idx);
     }
   }
@@ -115,8 +120,9 @@ greedy_finish_kernel(const bf16_t* __restrict__ logits, int V, int nc, int norma
 
 size_t greedy_scratch_floats(int T, int V) { return (size_t)T * 2 * ((V + 1023) / 1024); }
 
-int k_greedy(orn_ctx* ctx, cudaStream_t s, const bf16_t* logits, int T, int V, int normalize,
-             uint32_t* tokens, float* scratch) {
+namespace {
+template <typename TL>
+int launch_greedy(orn_ctx* ctx, cudaStream_t s, const TL* logits, int T, int V, int normalize, uint32_t* tokens, float* scratch) {
   const int nc = (V + 1023) / 1024;
   dim3 grid(nc, T);
   lse_chunk_kernel<<<grid, 256, 0, s>>>(logits, V, nc, scratch);
@@ -126,6 +132,16 @@ int k_greedy(orn_ctx* ctx, cudaStream_t s, const bf16_t* logits, int T, int V, i
   if (shm > 40000) ORN_FAIL(ctx, ORN_ERR_ARG, "greedy: vocabulary too large");
   greedy_finish_kernel<<<T, 256, shm, s>>>(logits, V, nc, normalize, scratch, tokens);
   return orn_launch_check(ctx, "greedy_finish");
+}
+}  // namespace
+
+int k_greedy(orn_ctx* ctx, cudaStream_t s, const bf16_t* logits, int T, int V, int normalize,
+             uint32_t* tokens, float* scratch) {
+  return launch_greedy(ctx, s, logits, T, V, normalize, tokens, scratch);
+}
+// float32 logits: the raw argmax, the lowest index winning ties
+int k_greedy_f32(orn_ctx* ctx, cudaStream_t s, const float* logits, int T, int V, uint32_t* tokens, float* scratch) {
+  return launch_greedy(ctx, s, logits, T, V, 0, tokens, scratch);
 }
 
 // ---------------------------------------------------------------------------
