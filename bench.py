@@ -777,6 +777,192 @@ def ours(args):
         dist.destroy_process_group()
 
 
+# ---- the Peratar decoder beside the Qwen3.5-MoE trunk at equal layer sizes
+PERATAR_SIZES = [  # width, heads, feed-forward, layers; head sizes and latent as real models have them
+    dict(width=1024, heads=8, ff=4096, layers=8, experts=(8, 4, 512, 768)),
+    dict(width=2048, heads=16, ff=8192, layers=8, experts=(8, 4, 1024, 1280)),
+    dict(width=4096, heads=32, ff=16384, layers=8, experts=None),  # above the trunk's fused kernels' hidden size
+]
+PERATAR_VOCAB = 32768
+
+
+def peratar_config(z, kv_rank=512, dim=128, rot=64, vdim=128):
+    """Three quarters of the layers own their cache, the last quarter reads the last owner's."""
+    own = z["layers"] * 3 // 4
+    ls = []
+    for i in range(z["layers"]):
+        mx = {"heads": z["heads"], "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": kv_rank, "scale": (dim + rot) ** -0.5,
+              "rot": {"base": 1e4, "dims": rot}}
+        if i >= own:
+            mx["kv_from"] = own - 1
+        ls.append({"type": "latent_attention", "mixer": mx, "mlp": {"kind": "dense", "ff": z["ff"]}})
+    return {"architecture": "Peratar", "width": z["width"], "vocab": PERATAR_VOCAB, "norm": {"eps": 1e-6}, "logit_softcap": 30.0,
+            "layers": ls}
+
+
+def trunk_of_equal_size(pkg, ctx, z, max_ctx):
+    """The trunk with attention in every layer and bf16 weights: about the same bytes per decoded token."""
+    E, k, inter, shared = z["experts"]
+    cfg = pkg.qwen35_config(max_ctx=max_ctx, hidden=z["width"], n_layers=z["layers"], full_attn_interval=1, n_heads=z["heads"],
+                            n_kv_heads=2, n_experts=E, top_k=k, expert_inter=inter, shared_inter=shared, vocab=PERATAR_VOCAB)
+    m = pkg.TextModel(ctx, cfg)
+    m.init_random(SEED)
+    H, QD, KVD = cfg.hidden, cfg.n_heads * cfg.head_dim, cfg.n_kv_heads * cfg.head_dim
+    shapes = {"self_attn.q_proj": (1, 2 * QD, H), "self_attn.k_proj": (1, KVD, H), "self_attn.v_proj": (1, KVD, H),
+              "self_attn.o_proj": (1, H, QD), "mlp.gate": (1, E, H), "mlp.switch_mlp.gate_proj": (E, inter, H),
+              "mlp.switch_mlp.up_proj": (E, inter, H), "mlp.switch_mlp.down_proj": (E, H, inter),
+              "mlp.shared_expert.gate_proj": (1, shared, H), "mlp.shared_expert.up_proj": (1, shared, H),
+              "mlp.shared_expert.down_proj": (1, H, shared), "mlp.shared_expert_gate": (1, 1, H)}
+    for i in range(cfg.n_layers):
+        for n, (e, o, kk) in shapes.items():
+            m.set_linear("layers.%d.%s" % (i, n), pkg.Linear.random(ctx, pkg.BF16, e, o, kk, SEED + 17 * i + o))
+    m.set_linear("lm_head", pkg.Linear.random(ctx, pkg.BF16, 1, PERATAR_VOCAB, H, SEED))
+    per_layer = 2 * (H * (2 * QD + 2 * KVD + QD + E + 1) + 3 * H * (k * inter + shared))
+    return m, cfg, cfg.n_layers * per_layer + 2 * PERATAR_VOCAB * H
+
+
+def peratar_label_work(z, cfg, label, T, ctx_len):
+    """(bytes, flops) a launch with this label has to move or compute: Peratar and trunk kernels alike."""
+    H, hs, w = z["heads"], 192, z["width"]
+    row, R, vd, dm = 576 * 2, 512, 128, 128
+    pairs = T * (T + 1) / 2
+    if label.startswith("decode_dense"):
+        O, K = (int(v) for v in label.split()[-1].split("x"))
+        return O * K * 2.0, 0
+    if label == "latent_attn":
+        return ctx_len * row + H * R * 4.0, 0
+    if label == "latent_absorb":
+        return H * dm * R * 2.0, 0
+    if label == "latent_out":
+        return H * vd * R * 2.0, 0
+    if label == "latent_flash":
+        return 0, 2.0 * H * pairs * (hs + vd)
+    if label == "flash_prefill":
+        return 0, 2.0 * H * pairs * 512
+    if label in ("k_attn", "k_attn_split"):
+        return ctx_len * 2 * 256 * 2 * 2.0, 0
+    if label.startswith("residual_rows"):
+        avg = (z["layers"] + 3) / 2 * 4 if "avg" in label else 0  # the streams an average reads, plus the one it writes
+        return T * w * (3 * 4 + 4 + 2 + avg), 0
+    if label == "add_rms_norm":
+        return T * w * 4 * 2.0, 0
+    if label == "latent_rows":
+        return T * (2 * H * 64 * 2 + 576 * 6.0), 0
+    if label.startswith("k_qgemm kind=3"):
+        f = dict(x.split("=") for x in label.split() if "=" in x)
+        plus, O, K, rows = "+" in f["O"], int(f["O"].rstrip("+")), int(f["K"]), int(f["rows"])
+        extra = {H * hs: 576 + H + w, z["ff"]: w, H * vd: H * dm} if plus else {}
+        return 0, 2.0 * (O + extra.get(O, 0)) * K * rows
+    if cfg is not None and len(label.split()) == 4 and "kind=3" in label:
+        b = peratar_trunk_bytes(cfg, label)
+        return (b, 0) if b else None
+    return None
+
+
+def peratar_trunk_bytes(cfg, label):
+    """Weight bytes of the trunk's fused decode launches with bf16 matrices."""
+    kern, _, _, shape = label.split()
+    O, K = (int(v) for v in shape.split("x"))
+    if kern == "k_moe_up":
+        return cfg.top_k * 2 * O * K * 2.0
+    if kern == "k_moe_down":
+        return (cfg.top_k * O * K + O * cfg.shared_inter) * 2.0
+    QD, KVD = cfg.n_heads * cfg.head_dim, cfg.n_kv_heads * cfg.head_dim
+    rows = O
+    if (O, K) == (2 * QD, cfg.hidden):
+        rows += 2 * KVD
+    elif (O, K) == (cfg.n_experts, cfg.hidden):
+        rows += 2 * cfg.shared_inter + 1
+    return rows * K * 2.0
+
+
+def peratar(args):
+    """Prefill and decode throughput of the Peratar decoder (random weights, whole public calls and device
+    time), its kernels against the measured peaks, and the trunk of equal size under the same clock."""
+    pkg = load_pkg()
+    ctx = pkg.Context(int(os.environ.get("LOCAL_RANK", "0")))
+    rng = np.random.default_rng(SEED)
+    hbm, which = peaks()
+    try:
+        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+            tf = json.load(f)["bf16_tflops"]
+    except (OSError, KeyError, ValueError):
+        tf = 1590.0
+    prompts, contexts, new = (512, 4096, 8192), (128, 8192), args.gen_tokens
+    max_ctx = max(prompts) + new + 64
+    ids = rng.integers(0, PERATAR_VOCAB, max(prompts)).astype(np.uint32)
+    sampler = ClockSampler(ctx.device)
+    sampler.start()
+    launches0 = ctx.launches()
+
+    def measure(model, token_bytes, z, cfg):
+        cache = model.make_cache()
+        out = {"bytes_per_token": token_bytes, "prefill": [], "decode": [], "kernels": []}
+        for T in prompts:
+            for _ in range(args.warmup):
+                cache.reset()
+                model.prefill(cache, ids[:T], 8192)
+            ctx.timer_start()
+            t0 = time.perf_counter()
+            for _ in range(args.steps):
+                cache.reset()
+                model.prefill(cache, ids[:T], 8192)
+            ms = ctx.timer_stop() / args.steps
+            wall = (time.perf_counter() - t0) / args.steps
+            out["prefill"].append({"tokens": T, "ms": ms, "tok_s": T / ms * 1e3, "e2e_tok_s": T / wall})
+        for C in contexts:
+            for i in range(args.warmup + args.steps):
+                if i == args.warmup:
+                    ms = wall = 0.0
+                cache.reset()
+                t0 = time.perf_counter()
+                pkg.generate_step(model, cache, ids[:C], new, 8192)
+                if i >= args.warmup:
+                    ms += model.prof().total_ms / args.steps
+                    wall += (time.perf_counter() - t0) / args.steps
+            out["decode"].append({"context": C, "us_per_token": ms * 1e3 / new, "tok_s": new / ms * 1e3, "e2e_tok_s": new / wall,
+                                  "weight_gbs": token_bytes / (ms / new) * 1e-6, "frac_hbm": token_bytes / (ms / new) * 1e-6 / hbm})
+        T = max(prompts)
+        cache.reset()
+        ctx.ktime_begin()
+        pkg.generate_step(model, cache, ids[:T], 16, 8192)
+        for label, (n, ms) in sorted(ctx.ktime_end().items(), key=lambda kv: -kv[1][1])[:24]:
+            work = peratar_label_work(z, cfg, label, T, T)
+            us = 1e3 * ms / n
+            k = {"kernel": label, "launches": n, "us": us}
+            if work is not None:
+                b, fl = work
+                k["bound"] = "tensor" if fl else "hbm"
+                k["frac"] = fl / us * 1e-6 / tf if fl else b / us * 1e-3 / hbm
+            out["kernels"].append(k)
+        cache.free()
+        return out
+
+    sizes = []
+    for z in PERATAR_SIZES:
+        m = pkg.TextModel.from_config(ctx, peratar_config(z), max_ctx=max_ctx)
+        m.init_random(SEED)
+        row = {"width": z["width"], "heads": z["heads"], "ff": z["ff"], "layers": z["layers"],
+               "peratar": measure(m, m.weight_bytes() - 2 * PERATAR_VOCAB * z["width"], z, None)}
+        m.free()
+        if z["experts"] is not None:
+            m, cfg, per_token = trunk_of_equal_size(pkg, ctx, z, max_ctx)
+            row["qwen3_5_moe_bf16"] = measure(m, per_token, z, cfg)
+            m.free()
+        sizes.append(row)
+    clocks = sampler.stop()
+    mid = sizes[1]["peratar"]["decode"][0]
+    emit({"metric": "Peratar decode throughput", "value": mid["tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
+          "warmup": args.warmup, "ms_per_step": mid["us_per_token"] * new * 1e-3, "higher_is_better": True, "scaling": "weak",
+          "vs_baseline": None, "dtype": "bf16 activations, f32 residual stream and accumulate", "data": "synthetic (random-init weights and ids)",
+          "config": {"workload": "width 2048, 16 heads, latent 512 + 64, ff 8192, 8 layers, 128-token prompt, %d greedy tokens" % new,
+                     "l2_policy": "weights read per token exceed L2 (126 MB)"},
+          "e2e": {"value": mid["e2e_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 128 * 4, "d2h_bytes_per_step": 4 * (new + 1)},
+          "gpu_launches": ctx.launches() - launches0, "clocks": clocks, "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": which},
+          "sizes": sizes})
+    ctx.close()
+
+
 def ep_layer(args):
     """Second workload (`--workload ep-layer`): one MoE decode layer in expert-parallel form at
     BASELINE config 5's decode width (64 sequences x verify width 2 = 128 rows in all, split evenly
@@ -922,8 +1108,9 @@ def main():
     ap.add_argument("--n-layers", type=int, default=40, help="fewer layers at the full layer sizes (profiling runs)")
     ap.add_argument("--long-prefill", action="store_true", help="run the 6621-token prefill leg at any layer count")
     ap.add_argument("--ep-decode", action="store_true", help="run the batched expert-parallel decode leg at any layer count")
-    ap.add_argument("--workload", default="decode", choices=["decode", "ep-layer"],
-                    help="decode: the MTP depth-1 decode loop (the headline); ep-layer: one expert-parallel MoE layer")
+    ap.add_argument("--workload", default="decode", choices=["decode", "ep-layer", "peratar"],
+                    help="decode: the MTP depth-1 decode loop (the headline); ep-layer: one expert-parallel MoE layer; "
+                         "peratar: prefill and decode of the Peratar decoder beside the trunk of equal size (1 GPU)")
     args = ap.parse_args()
     global GEN_TOKENS, PROMPT_LEN
     GEN_TOKENS, PROMPT_LEN = args.gen_tokens, args.prompt_len
@@ -931,6 +1118,8 @@ def main():
         reference(args)
     elif args.workload == "ep-layer":
         ep_layer(args)
+    elif args.workload == "peratar":
+        peratar(args)
     else:
         ours(args)
 

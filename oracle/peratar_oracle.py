@@ -44,11 +44,16 @@ def rotate_pairs(x, pos, base, dims):
     return out
 
 
+def rotate_part(x, pos, mx):
+    """The rotated part of a query or key under the mixer's own rotation (none when it is empty)."""
+    return rotate_pairs(x, pos, mx["rot"]["base"], mx["rot"]["dims"]) if mx["rot_dim"] else x
+
+
 def latent_kv(h, pos, w_dkv, w_norm, mx, eps):
     """-> (latent [T, kv_rank], shared rotated key part [T, rot_dim])."""
     y = h @ w_dkv.T
     r = mx["kv_rank"]
-    return rms_norm(y[:, :r], w_norm, eps), rotate_pairs(y[:, r:], pos, mx["rot"]["base"], mx["rot"]["dims"])
+    return rms_norm(y[:, :r], w_norm, eps), rotate_part(y[:, r:], pos, mx)
 
 
 def causal_softmax(s):
@@ -66,7 +71,7 @@ def latent_attention(h, c, kr, W, p, mx):
     T = h.shape[0]
     pos = np.arange(T)
     q = (h @ W[p + "q"].T).reshape(T, H, d + r)
-    qr = rotate_pairs(q[:, :, d:], pos, mx["rot"]["base"], mx["rot"]["dims"])
+    qr = rotate_part(q[:, :, d:], pos, mx)
     k = (c @ W[p + "uk"].T).reshape(T, H, d)
     val = (c @ W[p + "uv"].T).reshape(T, H, v)
     gate = sigmoid(h @ W[p + "g"].T)

@@ -198,6 +198,7 @@ __global__ void __launch_bounds__(256) linear_plain_kernel(LinDev L, const TA* _
 constexpr int kDecThreads = 256;
 constexpr int kDecWarps = kDecThreads / 32;
 constexpr size_t kDecSmemMax = 200 * 1024;
+constexpr int kDecRegs = 4;  // a residual row of up to kDecRegs * 1024 entries stays in registers
 
 struct DecJobDev {
   const uint8_t* w;
@@ -242,6 +243,64 @@ ORN_D void decode_prologue(const DecParams& P, bf16_t* s_x, float* s_f, float* r
         f[d] = v;
         if (lead) { p.x_out[(size_t)m * Kp + d] = v; p.stream_out[(size_t)m * Kp + d] = v; }
         xs[d] = f2bf(v);
+      }
+    } else if (Kp <= kDecRegs * 4 * kDecThreads) {
+      // everything the row needs is requested at once and stays in registers
+      const size_t base = (size_t)m * R.ld;
+      float z[kDecRegs][4], x[kDecRegs][4], pt[kDecRegs][4];
+      const float al = R.n_avg > 0 ? bf2f(R.a[R.n_avg - 1]) : 0.f;
+      uint32_t wq[kDecRegs][2];
+#pragma unroll
+      for (int it = 0; it < kDecRegs; ++it) {
+        const int d = 4 * (threadIdx.x + it * kDecThreads);
+        const bool in = d < Kp;
+        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+        const float4 y4 = in ? __ldcg(reinterpret_cast<const float4*>(R.y + base + d)) : zero;
+        const float4 g4 = in && R.gate != nullptr ? __ldcg(reinterpret_cast<const float4*>(R.gate + base + d)) : zero;
+        const float4 x4 = in ? __ldcg(reinterpret_cast<const float4*>(R.x_in + base + d)) : zero;
+        const float4 p4 = in && R.n_avg > 0 ? __ldcg(reinterpret_cast<const float4*>(p.part + base + d)) : zero;
+        float b[4] = {0.f, 0.f, 0.f, 0.f}, w[4] = {0.f, 0.f, 0.f, 0.f}, g[4];
+        if (in && R.gate != nullptr) load_bf4(R.gate_b, d, K, b);
+        if (in) load_bf4(R.w, d, K, w);
+        unpack4(y4, z[it]); unpack4(g4, g); unpack4(x4, x[it]); unpack4(p4, pt[it]);
+        wq[it][0] = (uint32_t)f2bf(w[0]) | ((uint32_t)f2bf(w[1]) << 16);  // exact: they are bf16
+        wq[it][1] = (uint32_t)f2bf(w[2]) | ((uint32_t)f2bf(w[3]) << 16);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          if (R.gate != nullptr) z[it][e] *= sigmoid_f32(g[e] + b[e]);
+          if (d + e >= K) z[it][e] = 0.f;
+        }
+      }
+      float sum = 0.f;
+#pragma unroll
+      for (int it = 0; it < kDecRegs; ++it)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sum += z[it][e];
+      const float mean = block_sum<kDecThreads>(sum, red) / (float)K;
+      float sq = 0.f;
+#pragma unroll
+      for (int it = 0; it < kDecRegs; ++it)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          if (4 * (int)(threadIdx.x + it * kDecThreads) + e < K) { const float c = z[it][e] - mean; sq = fmaf(c, c, sq); }
+      const float rstd = 1.0f / sqrtf(block_sum<kDecThreads>(sq, red) / (float)K + R.eps);
+#pragma unroll
+      for (int it = 0; it < kDecRegs; ++it) {
+        const int d = 4 * (threadIdx.x + it * kDecThreads);
+        if (d >= Kp) break;
+        const float w[4] = {__uint_as_float(wq[it][0] << 16), __uint_as_float(wq[it][0] & 0xffff0000u), __uint_as_float(wq[it][1] << 16),
+                            __uint_as_float(wq[it][1] & 0xffff0000u)};
+        float v[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[e] = d + e < K ? fmaf((z[it][e] - mean) * rstd, w[e], x[it][e]) : 0.f;
+        if (R.n_avg > 0) {
+          if (lead) *reinterpret_cast<float4*>(p.stream_out + base + d) = make_float4(v[0], v[1], v[2], v[3]);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) v[e] = fmaf(al, v[e], pt[it][e]);
+        }
+        if (lead) *reinterpret_cast<float4*>(p.x_out + base + d) = make_float4(v[0], v[1], v[2], v[3]);
+        if (p.w2 != nullptr) *reinterpret_cast<float4*>(f + d) = make_float4(v[0], v[1], v[2], v[3]);
+        store_act4(xs + d, v);
       }
     } else {
       const size_t base = (size_t)m * R.ld;
@@ -312,7 +371,7 @@ ORN_D float bfhi(uint32_t u) { return __uint_as_float(u & 0xffff0000u); }
 template <int M, int R, int U>
 __global__ void __launch_bounds__(kDecThreads) decode_dense_kernel(const __grid_constant__ DecParams P) {
   extern __shared__ __align__(16) uint8_t s_raw[];
-  __shared__ float red[33];
+  __shared__ float red[33], s_act[4][2];
   bf16_t* s_x = reinterpret_cast<bf16_t*>(s_raw);
   float* s_f = reinterpret_cast<float*>(s_raw + (((size_t)M * P.Kp * 2 + 15) & ~(size_t)15));
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -341,6 +400,7 @@ __global__ void __launch_bounds__(kDecThreads) decode_dense_kernel(const __grid_
     locate(task);
     load(0);
   }
+  if (threadIdx.x < P.njobs) act_prepare(P.job[threadIdx.x].act, s_act[threadIdx.x][0], s_act[threadIdx.x][1]);
   pdl_wait();
   pdl_trigger();
   decode_prologue<M>(P, s_x, s_f, red);
@@ -393,9 +453,7 @@ __global__ void __launch_bounds__(kDecThreads) decode_dense_kernel(const __grid_
         if (lane == r * M + m) { mine = acc[r][m]; mr = r; mm = m; }
     if (lane < R * M && oo + mr < J.O) {
       const int o = oo + mr;
-      float pa, pb;
-      act_prepare(J.act, pa, pb);
-      const float v = act_apply(J.act.kind, mine + (J.bias != nullptr ? bf2f(J.bias[o]) : 0.f), pa, pb);
+      const float v = act_apply(J.act.kind, mine + (J.bias != nullptr ? bf2f(J.bias[o]) : 0.f), s_act[jj][0], s_act[jj][1]);
       if (J.out_f32) reinterpret_cast<float*>(J.y)[(size_t)mm * J.ldy + o] = v;
       else reinterpret_cast<bf16_t*>(J.y)[(size_t)mm * J.ldy + o] = f2bf(v);
     }
@@ -497,9 +555,10 @@ int f_decode_dense(orn_ctx* ctx, cudaStream_t s, int M, const DecodePrologue& p,
     if (L->kind != ORN_BF16 || L->E != 1 || L->K != P.Kp) ORN_FAIL(ctx, ORN_ERR_ARG, "decode product: bf16 matrices over the staged rows");
     total += L->O;
   }
-  // rows per warp: two where that still gives every warp of the GPU a task
-  const long warps = 2L * ctx->sm_count * kDecWarps;
-  const int R = total >= 2 * warps ? 2 : 1;
+  const int fit = (int)std::max<size_t>(1, std::min<size_t>(2, (220 * 1024) / (smem + 2048)));
+  // rows per warp: two where that costs no extra round over the GPU's warps
+  const long warps = (long)fit * ctx->sm_count * kDecWarps;
+  const int R = 2 * ((total + 2 * warps - 1) / (2 * warps)) <= (total + warps - 1) / warps ? 2 : 1;
   P.tasks = 0;
   for (int j = 0; j < njobs; ++j) {
     DecJobDev& D = P.job[j];
@@ -508,7 +567,6 @@ int f_decode_dense(orn_ctx* ctx, cudaStream_t s, int M, const DecodePrologue& p,
     D.out_f32 = jobs[j].out_f32 ? 1 : 0; D.bias = jobs[j].bias; D.act = jobs[j].act;
     P.tasks += (L->O + R - 1) / R;
   }
-  const int fit = (int)std::max<size_t>(1, std::min<size_t>(2, (220 * 1024) / (smem + 2048)));
   const int grid = std::min((P.tasks + kDecWarps - 1) / kDecWarps, fit * ctx->sm_count);
   const char* label = "decode_dense";
   if (ctx->kt != nullptr) {  // per-kernel timing: one label per shape

@@ -92,10 +92,22 @@ __global__ void __launch_bounds__(kLrThreads) latent_absorb_kernel(LatentDims D,
   extern __shared__ float s_q[];  // [dim]
   __shared__ float s_part[4][kAbCols];
   __shared__ float red[4];
-  pdl_wait();
-  pdl_trigger();
   const int nq = T * D.heads * chunks;
   int b = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  // the head's first rows do not depend on the kernel before this one
+  constexpr int kPre = 16;
+  uint2 pre[kPre];
+  if (b < nq) {
+    const int h = (b / chunks) % D.heads, r0 = (b % chunks) * kAbCols + 4 * lane;
+#pragma unroll
+    for (int k = 0; k < kPre; ++k) {
+      const int i = warp + 4 * k;
+      pre[k] = i < D.dim && r0 < D.rp() ? __ldg(reinterpret_cast<const uint2*>(uk.w + (size_t)(h * D.dim + i) * uk.rec + 2 * (size_t)r0)) : make_uint2(0, 0);
+    }
+  }
+  pdl_wait();
+  pdl_trigger();
   if (b < nq) {
     const int c = b % chunks, h = (b / chunks) % D.heads, t = b / (chunks * D.heads);
     const TA* qr = q + (size_t)t * ldq + (size_t)h * D.qk();
@@ -108,19 +120,32 @@ __global__ void __launch_bounds__(kLrThreads) latent_absorb_kernel(LatentDims D,
         out[RP + i] = to_act<TA>(i < D.rot_dim ? rotated(i, D.rot_dims, p, D.freq, [&](int e) { return from_act(__ldcg(qr + D.dim + e)); }) : 0.f);
     }
     __syncthreads();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int r0 = c * kAbCols + 4 * lane;  // four latent entries per lane, a quarter of the head's rows per warp
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
     if (r0 < D.rp()) {
       const uint8_t* w = uk.w + (size_t)(h * D.dim) * uk.rec + 2 * (size_t)r0;
-#pragma unroll 8
-      for (int i = warp; i < D.dim; i += 4) {
-        const uint2 u = __ldg(reinterpret_cast<const uint2*>(w + (size_t)i * uk.rec));
-        const float x = s_q[i];
+      auto add = [&](const uint2& u, float x) {
         acc[0] = fmaf(x, __uint_as_float(u.x << 16), acc[0]);
         acc[1] = fmaf(x, __uint_as_float(u.x & 0xffff0000u), acc[1]);
         acc[2] = fmaf(x, __uint_as_float(u.y << 16), acc[2]);
         acc[3] = fmaf(x, __uint_as_float(u.y & 0xffff0000u), acc[3]);
+      };
+      uint2 nxt[kPre];  // the rows after those, all in flight before the first is used
+#pragma unroll
+      for (int k = 0; k < kPre; ++k) {
+        const int i = warp + 4 * (kPre + k);
+        nxt[k] = i < D.dim ? __ldg(reinterpret_cast<const uint2*>(w + (size_t)i * uk.rec)) : make_uint2(0, 0);
+      }
+#pragma unroll
+      for (int k = 0; k < kPre; ++k)
+        if (warp + 4 * k < D.dim) add(pre[k], s_q[warp + 4 * k]);
+#pragma unroll
+      for (int k = 0; k < kPre; ++k)
+        if (warp + 4 * (kPre + k) < D.dim) add(nxt[k], s_q[warp + 4 * (kPre + k)]);
+#pragma unroll 8
+      for (int i = warp + 8 * kPre; i < D.dim; i += 4) {
+        const uint2 u = __ldg(reinterpret_cast<const uint2*>(w + (size_t)i * uk.rec));
+        add(u, s_q[i]);
       }
     }
 #pragma unroll
@@ -359,19 +384,31 @@ __global__ void __launch_bounds__(kLaWarps * 32) latent_attn_kernel(LatentDims D
 }
 
 // ------------------------------------------------------------------ absorbed form: output
-constexpr int kLoThreads = 128, kLoRows = 32;  // value rows per CTA
+constexpr int kLoThreads = 256, kLoRows = 32;  // value rows per CTA
 template <typename TA>
-__global__ void __launch_bounds__(kLoThreads) latent_out_kernel(LatentDims D, int T, int cap, LinDev uv, const float* __restrict__ partial,
+__global__ void __launch_bounds__(kLoThreads) latent_out_kernel(LatentDims D, int T, LinDev uv, const float* __restrict__ partial,
                                                                 const float* __restrict__ ml, int splits, int plain,
                                                                 const int* __restrict__ pos, const float* __restrict__ gate, int ldgate,
                                                                 TA* __restrict__ att, int ldatt) {
-  extern __shared__ float s_c[];  // [rp] merged latent, then [splits] weights
+  extern __shared__ float s_c[];  // [rp] merged latent, [splits] weights, [8 * 32 * 4] partial sums of a merge pass
   __shared__ float s_tot;
-  pdl_wait();
-  pdl_trigger();
   const int R = D.kv_rank, RP = D.rp();
   const int rh = blockIdx.x, t = rh / D.heads, h = rh - t * D.heads;
-  float* s_w = s_c + RP;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int row0 = blockIdx.y * kLoRows + warp, row1 = min(D.vdim, (int)(blockIdx.y + 1) * kLoRows);
+  // the first pieces of this warp's value rows do not depend on the kernel before this one
+  constexpr int kPre = kLoRows / (kLoThreads / 32);
+  uint4 pre[kPre][2];
+#pragma unroll
+  for (int i = 0; i < kPre; ++i)
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int r = row0 + i * (kLoThreads / 32), c = lane + 32 * u;
+      pre[i][u] = r < row1 && c < RP / 8 ? ldg128(uv.w + (size_t)(h * D.vdim + r) * uv.rec + 16 * (size_t)c) : make_uint4(0, 0, 0, 0);
+    }
+  pdl_wait();
+  pdl_trigger();
+  float *s_w = s_c + RP, *s_m = s_w + ((splits + 3) & ~3);
   int used = 1;
   if (!plain) {
     const int n = *pos + T;
@@ -379,48 +416,63 @@ __global__ void __launch_bounds__(kLoThreads) latent_out_kernel(LatentDims D, in
     used = min(splits, (n + kps - 1) / kps);
   }
   const float* mlr = ml + 2 * (size_t)rh * splits;
-  if (threadIdx.x < 32) {
+  if (warp == 0) {
     float m = -INFINITY;
-    for (int i = threadIdx.x; i < used; i += 32) m = fmaxf(m, __ldcg(mlr + 2 * i));
+    for (int i = lane; i < used; i += 32) m = fmaxf(m, __ldcg(mlr + 2 * i));
     m = warp_max(m);
     float tot = 0.f;
-    for (int i = threadIdx.x; i < used; i += 32) {
+    for (int i = lane; i < used; i += 32) {
       const float w = exp2f(__ldcg(mlr + 2 * i) - m);
       s_w[i] = w;
       tot = fmaf(w, __ldcg(mlr + 2 * i + 1), tot);
     }
     tot = warp_sum(tot);
-    if (threadIdx.x == 0) s_tot = tot;
+    if (lane == 0) s_tot = tot;
   }
   __syncthreads();
   const float inv = 1.0f / s_tot;
-  for (int i = threadIdx.x; i < RP; i += kLoThreads) {
-    float a = 0.f;
-    if (i < R) {
+  // 32 float4 columns per pass, the splits dealt to the warps; a fixed order of additions
+  const float* pr = partial + (size_t)rh * splits * R;
+  for (int c0 = 0; c0 < RP; c0 += 128) {
+    const int i = c0 + 4 * lane;
+    float a[4] = {0.f, 0.f, 0.f, 0.f};
+    if (i + 3 < R && (R & 3) == 0) {
 #pragma unroll 8
-      for (int sp = 0; sp < used; ++sp) {
+      for (int sp = warp; sp < used; sp += kLoThreads / 32) {
         const float w = s_w[sp];
-        if (w != 0.f) a = fmaf(w, __ldcg(partial + ((size_t)rh * splits + sp) * R + i), a);
+        const float4 v = __ldcg(reinterpret_cast<const float4*>(pr + (size_t)sp * R + i));
+        a[0] = fmaf(w, v.x, a[0]); a[1] = fmaf(w, v.y, a[1]); a[2] = fmaf(w, v.z, a[2]); a[3] = fmaf(w, v.w, a[3]);
       }
+    } else {
+      for (int sp = warp; sp < used; sp += kLoThreads / 32)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          if (i + e < R) a[e] = fmaf(s_w[sp], __ldcg(pr + (size_t)sp * R + i + e), a[e]);
     }
-    a *= inv;
-    s_c[i] = a;
+    *reinterpret_cast<float4*>(s_m + 128 * warp + 4 * lane) = make_float4(a[0], a[1], a[2], a[3]);
+    __syncthreads();
+    if (threadIdx.x < 128 && c0 + threadIdx.x < RP) {
+      float v = 0.f;
+#pragma unroll
+      for (int w = 0; w < kLoThreads / 32; ++w) v += s_m[128 * w + threadIdx.x];
+      s_c[c0 + threadIdx.x] = c0 + (int)threadIdx.x < R ? v * inv : 0.f;
+    }
+    __syncthreads();
   }
-  __syncthreads();
   const float gt = sigmoid_f32(__ldcg(gate + (size_t)t * ldgate + h));
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int i1 = min(D.vdim, (int)(blockIdx.y + 1) * kLoRows);
-#pragma unroll 2
-  for (int i = blockIdx.y * kLoRows + warp; i < i1; i += kLoThreads / 32) {
+#pragma unroll
+  for (int k = 0; k < kPre; ++k) {
+    const int i = row0 + k * (kLoThreads / 32);
+    if (i >= row1) break;  // warp-uniform
     const uint8_t* w = uv.w + (size_t)(h * D.vdim + i) * uv.rec;
     float a = 0.f;
-    for (int c = lane; c < RP / 8; c += 32) {
-      const uint4 u = ldg128(w + 16 * (size_t)c);
+    for (int c = lane, u = 0; c < RP / 8; c += 32, ++u) {
+      const uint4 v = u == 0 ? pre[k][0] : u == 1 ? pre[k][1] : ldg128(w + 16 * (size_t)c);
       const float4 x = *reinterpret_cast<const float4*>(s_c + 8 * c), y = *reinterpret_cast<const float4*>(s_c + 8 * c + 4);
-      a = fmaf(__uint_as_float(u.x << 16), x.x, a); a = fmaf(__uint_as_float(u.x & 0xffff0000u), x.y, a);
-      a = fmaf(__uint_as_float(u.y << 16), x.z, a); a = fmaf(__uint_as_float(u.y & 0xffff0000u), x.w, a);
-      a = fmaf(__uint_as_float(u.z << 16), y.x, a); a = fmaf(__uint_as_float(u.z & 0xffff0000u), y.y, a);
-      a = fmaf(__uint_as_float(u.w << 16), y.z, a); a = fmaf(__uint_as_float(u.w & 0xffff0000u), y.w, a);
+      a = fmaf(__uint_as_float(v.x << 16), x.x, a); a = fmaf(__uint_as_float(v.x & 0xffff0000u), x.y, a);
+      a = fmaf(__uint_as_float(v.y << 16), x.z, a); a = fmaf(__uint_as_float(v.y & 0xffff0000u), x.w, a);
+      a = fmaf(__uint_as_float(v.z << 16), y.x, a); a = fmaf(__uint_as_float(v.z & 0xffff0000u), y.y, a);
+      a = fmaf(__uint_as_float(v.w << 16), y.z, a); a = fmaf(__uint_as_float(v.w & 0xffff0000u), y.w, a);
     }
     a = warp_sum(a);
     if (lane == 0) att[(size_t)t * ldatt + (size_t)h * D.vdim + i] = to_act<TA>(a * gt);
@@ -428,7 +480,8 @@ __global__ void __launch_bounds__(kLoThreads) latent_out_kernel(LatentDims D, in
 }
 
 // ------------------------------------------------------------------ expanded form
-constexpr int kLfWarps = 4, kLfRows = 16 * kLfWarps, kLfKeys = 64;
+constexpr int kLfWarps = 4, kLfRows = 16 * kLfWarps, kLfKeys = 32;
+constexpr int kLfTiles = kLfKeys / 8;  // 8-key accumulator tiles per stage
 
 struct FlashArgs {
   const bf16_t *q, *kx, *vx, *cache;
@@ -442,7 +495,7 @@ struct FlashArgs {
 };
 
 template <int NV>  // 16-column groups of the value
-__global__ void __launch_bounds__(kLfWarps * 32) latent_flash_kernel(LatentDims D, FlashArgs A) {
+__global__ void __launch_bounds__(kLfWarps * 32, NV <= 8 ? 3 : 2) latent_flash_kernel(LatentDims D, FlashArgs A) {
   extern __shared__ __align__(128) uint8_t fsm[];
   const int qt = gridDim.x - 1 - blockIdx.x;  // the tiles with the most keys start first
   const int h = blockIdx.y;
@@ -496,15 +549,15 @@ __global__ void __launch_bounds__(kLfWarps * 32) latent_flash_kernel(LatentDims 
     const uint32_t kt = st_s + (i & 1) * stage, vt = kt + kLfKeys * kB;
     const int n0 = i * kLfKeys;
     if (n0 <= wlast) {  // warp-uniform: otherwise every key of this tile is in the future of every row
-      float s[8][4];
+      float s[kLfTiles][4];
 #pragma unroll
-      for (int j = 0; j < 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
+      for (int j = 0; j < kLfTiles; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
 #pragma unroll 4
       for (int kk = 0; kk < A.kd / 16; ++kk) {
         uint32_t a[4];
         ldsm4(q_s + a_off + 32 * kk, a);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
+        for (int j = 0; j < kLfTiles / 2; ++j) {
           uint32_t b[4];
           ldsm4(kt + k_off + j * 16 * kB + 32 * kk, b);
           mma16816(s[2 * j], a, b[0], b[1]);
@@ -512,28 +565,31 @@ __global__ void __launch_bounds__(kLfWarps * 32) latent_flash_kernel(LatentDims 
         }
       }
       const bool all_visible = n0 + kLfKeys <= p0 + wrow + 1 && n0 + kLfKeys <= n;
+      if (!all_visible) {
+#pragma unroll
+        for (int j = 0; j < kLfTiles; ++j)
+#pragma unroll
+          for (int c = 0; c < 4; ++c)
+            if (n0 + 8 * j + 2 * qd + (c & 1) >= min(n, c < 2 ? lim0 : lim1)) s[j][c] = -INFINITY;
+      }
       float x0 = -INFINITY, x1 = -INFINITY;
 #pragma unroll
-      for (int j = 0; j < 8; ++j)
-#pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          const int key = n0 + 8 * j + 2 * qd + (c & 1);
-          const float v = s[j][c] * sc2;
-          s[j][c] = (all_visible || key < min(n, c < 2 ? lim0 : lim1)) ? v : -INFINITY;
-          if (c < 2) x0 = fmaxf(x0, s[j][c]);
-          else x1 = fmaxf(x1, s[j][c]);
-        }
+      for (int j = 0; j < kLfTiles; ++j) {
+        x0 = fmaxf(x0, fmaxf(s[j][0], s[j][1]));
+        x1 = fmaxf(x1, fmaxf(s[j][2], s[j][3]));
+      }
       x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 1)); x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 2));
       x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 1)); x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 2));
-      const float a0 = fmaxf(m0, x0), a1 = fmaxf(m1, x1);
+      // maxima in the scaled domain (the scale is positive here)
+      const float a0 = fmaxf(m0, x0 * sc2), a1 = fmaxf(m1, x1 * sc2);
       const float u0 = a0 == -INFINITY ? 0.f : a0, u1 = a1 == -INFINITY ? 0.f : a1;
       const float c0 = exp2f(m0 - u0), c1 = exp2f(m1 - u1);
       m0 = a0; m1 = a1;
       float t0 = 0.f, t1 = 0.f;
 #pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        s[j][0] = exp2f(s[j][0] - u0); s[j][1] = exp2f(s[j][1] - u0);
-        s[j][2] = exp2f(s[j][2] - u1); s[j][3] = exp2f(s[j][3] - u1);
+      for (int j = 0; j < kLfTiles; ++j) {
+        s[j][0] = exp2f(fmaf(s[j][0], sc2, -u0)); s[j][1] = exp2f(fmaf(s[j][1], sc2, -u0));
+        s[j][2] = exp2f(fmaf(s[j][2], sc2, -u1)); s[j][3] = exp2f(fmaf(s[j][3], sc2, -u1));
         t0 += s[j][0] + s[j][1];
         t1 += s[j][2] + s[j][3];
       }
@@ -544,7 +600,7 @@ __global__ void __launch_bounds__(kLfWarps * 32) latent_flash_kernel(LatentDims 
         for (int j = 0; j < 2 * NV; ++j) { o[j][0] *= c0; o[j][1] *= c0; o[j][2] *= c1; o[j][3] *= c1; }
       }
 #pragma unroll
-      for (int ks = 0; ks < 4; ++ks) {
+      for (int ks = 0; ks < kLfKeys / 16; ++ks) {
         const uint32_t pa[4] = {pack_bf16x2(s[2 * ks][0], s[2 * ks][1]), pack_bf16x2(s[2 * ks][2], s[2 * ks][3]),
                                 pack_bf16x2(s[2 * ks + 1][0], s[2 * ks + 1][1]), pack_bf16x2(s[2 * ks + 1][2], s[2 * ks + 1][3])};
 #pragma unroll
@@ -664,20 +720,20 @@ int k_latent_attn(orn_ctx* ctx, cudaStream_t s, const LatentDims& D, int T, cons
 int k_latent_out(orn_ctx* ctx, cudaStream_t s, const LatentDims& D, int T, const orn_linear* uv, const float* partial, const float* ml,
                  int splits, const int* pos, const float* gate, int ldgate, void* att, int ldatt, bool plain, bool act_f32) {
   const dim3 grid(T * D.heads, (D.vdim + kLoRows - 1) / kLoRows);
-  const size_t smem = sizeof(float) * (size_t)(D.rp() + splits);
-  if (smem > 48 * 1024) ORN_FAIL(ctx, ORN_ERR_ARG, "latent attention: latent above 12000 entries");
+  const size_t smem = sizeof(float) * (size_t)(D.rp() + ((splits + 3) & ~3) + 128 * (kLoThreads / 32));
+  if (smem > 48 * 1024) ORN_FAIL(ctx, ORN_ERR_ARG, "latent attention: latent above 11000 entries");
   if (act_f32)
-    ORN_CHECK_CUDA(ctx, orn_launch_dependent(ctx, s, 0, latent_out_kernel<float>, grid, dim3(kLoThreads), smem, D, T, 0, lin_dev(uv), partial, ml, splits,
+    ORN_CHECK_CUDA(ctx, orn_launch_dependent(ctx, s, 0, latent_out_kernel<float>, grid, dim3(kLoThreads), smem, D, T, lin_dev(uv), partial, ml, splits,
                                              plain ? 1 : 0, pos, gate, ldgate, (float*)att, ldatt));
   else
-    ORN_CHECK_CUDA(ctx, orn_launch_dependent(ctx, s, 0, latent_out_kernel<bf16_t>, grid, dim3(kLoThreads), smem, D, T, 0, lin_dev(uv), partial, ml, splits,
+    ORN_CHECK_CUDA(ctx, orn_launch_dependent(ctx, s, 0, latent_out_kernel<bf16_t>, grid, dim3(kLoThreads), smem, D, T, lin_dev(uv), partial, ml, splits,
                                              plain ? 1 : 0, pos, gate, ldgate, (bf16_t*)att, ldatt));
   return orn_launch_check(ctx, "latent_out");
 }
 
 bool latent_flash_ok(const LatentDims& D, int ldq) {
   const int kd = (D.qk() + 15) & ~15, vd = (D.vdim + 15) & ~15;
-  return D.dim % 8 == 0 && D.rot_dim % 8 == 0 && D.vdim % 8 == 0 && ldq % 8 == 0 && D.vdim <= 256 && latent_flash_smem(D, kd, vd) <= kSmemMax;
+  return D.scale > 0.f && D.dim % 8 == 0 && D.rot_dim % 8 == 0 && D.vdim % 8 == 0 && ldq % 8 == 0 && D.vdim <= 256 && latent_flash_smem(D, kd, vd) <= kSmemMax;
 }
 
 int k_latent_flash(orn_ctx* ctx, cudaStream_t s, const LatentDims& D, int T, const bf16_t* q, int ldq, const bf16_t* kx, int ldk, const bf16_t* vx,
