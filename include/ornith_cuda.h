@@ -334,7 +334,7 @@ int32_t orn_model_create_json(orn_ctx* ctx, const char* config_json, int32_t max
  * among these tokens (n_want may be 0).  Serves every architecture of the registry. */
 int32_t orn_step(orn_model* m, orn_cache* c, const uint32_t* host_ids, int32_t n, int32_t prefill_step,
                  const int32_t* host_want, int32_t n_want, float* dev_logits);
-/* a checker's view of the layers: during every later orn_step of n tokens dev_tap [layers, n, hidden]
+/* a view into the layers, for tests: during every later orn_step of n tokens dev_tap [layers, n, hidden]
  * receives the float32 stream after each layer (NULL: off).  Registered decoders only; windows then run
  * without CUDA graphs. */
 int32_t orn_model_tap(orn_model* m, float* dev_tap);

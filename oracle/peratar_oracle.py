@@ -1,6 +1,6 @@
 """Plain restatement of the Peratar decoder in numpy, one function per mechanism.
 
-The checker of csrc/decoder.cu and its kernels: slow, whole sequence at once, float64 unless asked
+What the tests hold csrc/decoder.cu and its kernels to: slow, whole sequence at once, float64 unless asked
 otherwise, no cache and no batching.  It shares no code with the product path.  `W` is a dict from
 tensor names to float arrays, `cfg` the parsed config.json.
 

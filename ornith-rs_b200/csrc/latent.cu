@@ -385,12 +385,13 @@ __global__ void __launch_bounds__(kLaWarps * 32) latent_attn_kernel(LatentDims D
 
 // ------------------------------------------------------------------ absorbed form: output
 constexpr int kLoThreads = 256, kLoRows = 32;  // value rows per CTA
+constexpr int kLoCols = 512;                   // latent columns per merge pass
 template <typename TA>
 __global__ void __launch_bounds__(kLoThreads) latent_out_kernel(LatentDims D, int T, LinDev uv, const float* __restrict__ partial,
                                                                 const float* __restrict__ ml, int splits, int plain,
                                                                 const int* __restrict__ pos, const float* __restrict__ gate, int ldgate,
                                                                 TA* __restrict__ att, int ldatt) {
-  extern __shared__ float s_c[];  // [rp] merged latent, [splits] weights, [8 * 32 * 4] partial sums of a merge pass
+  extern __shared__ float s_c[];  // [rp] merged latent, [splits] weights, [warps][kLoCols] partial sums of a merge pass
   __shared__ float s_tot;
   const int R = D.kv_rank, RP = D.rp();
   const int rh = blockIdx.x, t = rh / D.heads, h = rh - t * D.heads;
@@ -431,31 +432,45 @@ __global__ void __launch_bounds__(kLoThreads) latent_out_kernel(LatentDims D, in
   }
   __syncthreads();
   const float inv = 1.0f / s_tot;
-  // 32 float4 columns per pass, the splits dealt to the warps; a fixed order of additions
+  // 512 columns per pass, the splits dealt to the warps; a fixed order of additions
   const float* pr = partial + (size_t)rh * splits * R;
-  for (int c0 = 0; c0 < RP; c0 += 128) {
-    const int i = c0 + 4 * lane;
-    float a[4] = {0.f, 0.f, 0.f, 0.f};
-    if (i + 3 < R && (R & 3) == 0) {
-#pragma unroll 8
+  for (int c0 = 0; c0 < RP; c0 += kLoCols) {
+    float a[4][4] = {};
+    if ((R & 3) == 0) {
+#pragma unroll 4
       for (int sp = warp; sp < used; sp += kLoThreads / 32) {
         const float w = s_w[sp];
-        const float4 v = __ldcg(reinterpret_cast<const float4*>(pr + (size_t)sp * R + i));
-        a[0] = fmaf(w, v.x, a[0]); a[1] = fmaf(w, v.y, a[1]); a[2] = fmaf(w, v.z, a[2]); a[3] = fmaf(w, v.w, a[3]);
+        float4 v[4];
+#pragma unroll
+        for (int g = 0; g < 4; ++g) {
+          const int i = c0 + 128 * g + 4 * lane;
+          v[g] = i < R ? __ldcg(reinterpret_cast<const float4*>(pr + (size_t)sp * R + i)) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int g = 0; g < 4; ++g) {
+          a[g][0] = fmaf(w, v[g].x, a[g][0]); a[g][1] = fmaf(w, v[g].y, a[g][1]);
+          a[g][2] = fmaf(w, v[g].z, a[g][2]); a[g][3] = fmaf(w, v[g].w, a[g][3]);
+        }
       }
     } else {
       for (int sp = warp; sp < used; sp += kLoThreads / 32)
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-          if (i + e < R) a[e] = fmaf(s_w[sp], __ldcg(pr + (size_t)sp * R + i + e), a[e]);
+        for (int g = 0; g < 4; ++g)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int i = c0 + 128 * g + 4 * lane + e;
+            if (i < R) a[g][e] = fmaf(s_w[sp], __ldcg(pr + (size_t)sp * R + i), a[g][e]);
+          }
     }
-    *reinterpret_cast<float4*>(s_m + 128 * warp + 4 * lane) = make_float4(a[0], a[1], a[2], a[3]);
+#pragma unroll
+    for (int g = 0; g < 4; ++g)
+      *reinterpret_cast<float4*>(s_m + kLoCols * warp + 128 * g + 4 * lane) = make_float4(a[g][0], a[g][1], a[g][2], a[g][3]);
     __syncthreads();
-    if (threadIdx.x < 128 && c0 + threadIdx.x < RP) {
+    for (int i = threadIdx.x; i < kLoCols && c0 + i < RP; i += kLoThreads) {
       float v = 0.f;
 #pragma unroll
-      for (int w = 0; w < kLoThreads / 32; ++w) v += s_m[128 * w + threadIdx.x];
-      s_c[c0 + threadIdx.x] = c0 + (int)threadIdx.x < R ? v * inv : 0.f;
+      for (int w = 0; w < kLoThreads / 32; ++w) v += s_m[kLoCols * w + i];
+      s_c[c0 + i] = c0 + i < R ? v * inv : 0.f;
     }
     __syncthreads();
   }
@@ -720,8 +735,8 @@ int k_latent_attn(orn_ctx* ctx, cudaStream_t s, const LatentDims& D, int T, cons
 int k_latent_out(orn_ctx* ctx, cudaStream_t s, const LatentDims& D, int T, const orn_linear* uv, const float* partial, const float* ml,
                  int splits, const int* pos, const float* gate, int ldgate, void* att, int ldatt, bool plain, bool act_f32) {
   const dim3 grid(T * D.heads, (D.vdim + kLoRows - 1) / kLoRows);
-  const size_t smem = sizeof(float) * (size_t)(D.rp() + ((splits + 3) & ~3) + 128 * (kLoThreads / 32));
-  if (smem > 48 * 1024) ORN_FAIL(ctx, ORN_ERR_ARG, "latent attention: latent above 11000 entries");
+  const size_t smem = sizeof(float) * (size_t)(D.rp() + ((splits + 3) & ~3) + kLoCols * (kLoThreads / 32));
+  if (smem > 48 * 1024) ORN_FAIL(ctx, ORN_ERR_ARG, "latent attention: latent above 8000 entries");
   if (act_f32)
     ORN_CHECK_CUDA(ctx, orn_launch_dependent(ctx, s, 0, latent_out_kernel<float>, grid, dim3(kLoThreads), smem, D, T, lin_dev(uv), partial, ml, splits,
                                              plain ? 1 : 0, pos, gate, ldgate, (float*)att, ldatt));
