@@ -14,6 +14,13 @@ struct ActParams {
 };
 
 #ifdef __CUDACC__
+// the activation type of a model: float32 or bfloat16
+template <typename T> __device__ __forceinline__ T to_act(float v);
+template <> __device__ __forceinline__ float to_act<float>(float v) { return v; }
+template <> __device__ __forceinline__ bf16_t to_act<bf16_t>(float v) { return f2bf(v); }
+ORN_D float from_act(float v) { return v; }
+ORN_D float from_act(bf16_t v) { return bf2f(v); }
+
 ORN_D float act_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 // the two scalars an activation needs, once per thread
 ORN_D void act_prepare(const ActParams& A, float& a, float& b) {

@@ -71,7 +71,7 @@ struct orn_decoder {
   bf16_t* final_norm = nullptr;
   orn_linear* head = nullptr;
   std::vector<float*> freq;  // per layer
-  int ldD = 0, ldq = 0, ldkv = 0, ldg = 0, ldatt = 0, ldu = 0, ldqa = 0;
+  int ldD = 0, ldq = 0, ldkv = 0, ldg = 0, ldatt = 0, ldu = 0;
   Scratch win, wide;         // windows (its addresses are in captured graphs); prompt chunks
   bf16_t *kx = nullptr, *vx = nullptr;  // expanded keys and values of one layer
   int exp_rows = 0, ldkx = 0, ldvx = 0;
@@ -389,7 +389,7 @@ int peratar_finalize(orn_model* m) {
   for (float* p : d->freq) cudaFree(p);
   d->freq.clear();
   d->ldD = pad8(s.width);
-  d->ldkv = d->ldg = d->ldq = d->ldatt = d->ldqa = 8;
+  d->ldkv = d->ldg = d->ldq = d->ldatt = 8;
   d->ldu = d->ldkx = d->ldvx = 8;
   for (size_t i = 0; i < s.layers.size(); ++i) {
     const std::string p = "l" + std::to_string(i) + ".";

@@ -30,12 +30,6 @@ ORN_D float block_sum(float v, float* red) {
   return t;
 }
 
-template <typename T> ORN_D T to_act(float v);
-template <> ORN_D float to_act<float>(float v) { return v; }
-template <> ORN_D bf16_t to_act<bf16_t>(float v) { return f2bf(v); }
-ORN_D float from_act(float v) { return v; }
-ORN_D float from_act(bf16_t v) { return bf2f(v); }
-
 ORN_D void store_act4(float* p, const float* v) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
 ORN_D void store_act4(bf16_t* p, const float* v) {
   uint2 u;
@@ -54,6 +48,9 @@ ORN_D void load_bf4(const bf16_t* p, int d, int width, float* v) {
   }
 }
 ORN_D void unpack4(const float4& f, float* v) { v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
+
+ORN_D float bflo(uint32_t u) { return __uint_as_float(u << 16); }
+ORN_D float bfhi(uint32_t u) { return __uint_as_float(u & 0xffff0000u); }
 
 // ------------------------------------------------------------------ row kernels
 constexpr int kRowThreads = 256;
@@ -237,12 +234,20 @@ ORN_D void decode_prologue(const DecParams& P, bf16_t* s_x, float* s_f, float* r
     bf16_t* xs = s_x + (size_t)m * Kp;
     if (p.mode == DRO_EMBED) {
       const uint32_t id = min(p.ids[m], (uint32_t)(P.table.O - 1));
-      const bf16_t* row = reinterpret_cast<const bf16_t*>(P.table.w + (size_t)id * P.table.rec);
-      for (int d = threadIdx.x; d < Kp; d += kDecThreads) {
-        const float v = d < K ? bf2f(row[d]) : 0.f;
-        f[d] = v;
-        if (lead) { p.x_out[(size_t)m * Kp + d] = v; p.stream_out[(size_t)m * Kp + d] = v; }
-        xs[d] = f2bf(v);
+      const uint8_t* row = P.table.w + (size_t)id * P.table.rec;  // padded with zeros to Kp
+      for (int c = threadIdx.x; c < Kp / 8; c += kDecThreads) {
+        const uint4 u = ldg128(row + 16 * (size_t)c);
+        const float4 lo = make_float4(bflo(u.x), bfhi(u.x), bflo(u.y), bfhi(u.y)), hi = make_float4(bflo(u.z), bfhi(u.z), bflo(u.w), bfhi(u.w));
+        const size_t at = (size_t)m * Kp + 8 * c;
+        *reinterpret_cast<uint4*>(xs + 8 * c) = u;
+        *reinterpret_cast<float4*>(f + 8 * c) = lo;
+        *reinterpret_cast<float4*>(f + 8 * c + 4) = hi;
+        if (lead) {
+          *reinterpret_cast<float4*>(p.x_out + at) = lo;
+          *reinterpret_cast<float4*>(p.x_out + at + 4) = hi;
+          *reinterpret_cast<float4*>(p.stream_out + at) = lo;
+          *reinterpret_cast<float4*>(p.stream_out + at + 4) = hi;
+        }
       }
     } else if (Kp <= kDecRegs * 4 * kDecThreads) {
       // everything the row needs is requested at once and stays in registers
@@ -363,9 +368,6 @@ ORN_D void decode_prologue(const DecParams& P, bf16_t* s_x, float* s_f, float* r
     __syncthreads();  // f is reused by the next row
   }
 }
-
-ORN_D float bflo(uint32_t u) { return __uint_as_float(u << 16); }
-ORN_D float bfhi(uint32_t u) { return __uint_as_float(u & 0xffff0000u); }
 
 // A warp takes R consecutive rows of one matrix: 32 lanes x 16 bytes per step and row, U steps in flight.
 template <int M, int R, int U>

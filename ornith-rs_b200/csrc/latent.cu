@@ -20,12 +20,6 @@
 
 namespace {
 
-template <typename T> ORN_D T to_act(float v);
-template <> ORN_D float to_act<float>(float v) { return v; }
-template <> ORN_D bf16_t to_act<bf16_t>(float v) { return f2bf(v); }
-ORN_D float from_act(float v) { return v; }
-ORN_D float from_act(bf16_t v) { return bf2f(v); }
-
 constexpr float kLog2e = 1.4426950408889634f;
 
 // entry i of a rotated vector v of n entries, the first `dims` in neighbouring pairs

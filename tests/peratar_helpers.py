@@ -44,8 +44,9 @@ CONFIGS = {
                              layer(mixer(1, 12, 2, 5, 11), None)], eps=1e-3, softcap=5.0),
     # one of everything
     "one": config(64, 70, [layer(mixer(1, 8, 2, 8, 8, base=3.0), 8)], softcap=2.0),
-    # no rotated part at all; only part of the rotated dimensions turn
-    "unrotated": config(72, 90, [layer(mixer(2, 16, 0, 16, 24), 40), layer(mixer(3, 8, 16, 16, 24, rot_dims=6), 40)]),
+    # no rotated part at all; only part of the rotated dimensions turn; the first layers have no feed-forward
+    "unrotated": config(72, 90, [layer(mixer(2, 16, 0, 16, 24), None), layer(mixer(1, 8, 8, 8, 16), None),
+                                 layer(mixer(3, 8, 16, 16, 24, rot_dims=6), 40)]),
     # a real layer's head sizes, more than sixteen heads
     "wide": config(512, 1000, [layer(mixer(20, 128, 64, 128, 512), 1024), layer(mixer(17, 128, 64, 128, 512, kv_from=0), 520)]),
     # latent and value widths at the ends of the tensor kernels' ranges
