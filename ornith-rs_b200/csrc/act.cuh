@@ -3,7 +3,7 @@
 
 #include "orn_common.cuh"
 
-enum { ACT_NONE = 0, ACT_XIELU = 1, ACT_SOFTCAP = 2 };
+enum { ACT_NONE = 0, ACT_XIELU = 1, ACT_SOFTCAP = 2, ACT_SILU = 3, ACT_SIGMOID = 4, ACT_GELU_TANH = 5 };
 
 // xIELU with the two learned numbers (p, q): a = softplus(p) scales the square above zero,
 // b = 1/2 + softplus(q) the exponential below; the slope at zero is 1/2 on both sides.
@@ -30,10 +30,15 @@ ORN_D void act_prepare(const ActParams& A, float& a, float& b) {
     b = 0.5f + act_softplus(bf2f(A.pq[1]));
   }
 }
+ORN_D float sigmoid_f32(float z) { return 1.0f / (1.0f + expf(-z)); }
+// z / 2 (1 + tanh u), u = sqrt(2 / pi) (z + 0.044715 z^3)
+ORN_D float gelu_tanh_f32(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z))); }
 ORN_D float act_apply(int kind, float z, float a, float b) {
   if (kind == ACT_XIELU) return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, expm1f(z) - z, 0.5f * z);
   if (kind == ACT_SOFTCAP) return a * tanhf(z / a);
+  if (kind == ACT_SILU) return z * sigmoid_f32(z);
+  if (kind == ACT_SIGMOID) return sigmoid_f32(z);
+  if (kind == ACT_GELU_TANH) return gelu_tanh_f32(z);
   return z;
 }
-ORN_D float sigmoid_f32(float z) { return 1.0f / (1.0f + expf(-z)); }
 #endif

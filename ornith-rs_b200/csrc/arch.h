@@ -39,3 +39,4 @@ const orn_arch* orn_arch_of_config(const orna::JVal& cfg);
 int qwen35_load(orn_ctx* ctx, const std::string& dir, const orna::JVal& cfg, int max_ctx, int dtype, orn_model** out);
 // decoder.cu
 extern const orn_arch kArchPeratar;
+extern const orn_arch kArchDokulorn;

@@ -57,10 +57,11 @@ size_t qgemm_scratch_bytes(int rows, int E, int O);
 int f_qgemm(orn_ctx* ctx, cudaStream_t s, const orn_linear* L, const bf16_t* x, int rows, void* y, int ldy,
             const QGemmGroup* grp /*nullable: dense*/, void* scratch /*grouped only*/, int out_f32 = 0,
             int bn_force = 0 /*> 0: token-tile width (multiple of 16, <= 256)*/);
-// what a bf16-weight product does to a result before storing it: y = act(x W^T + bias)
+// what a bf16-weight product does to a result before storing it: y = act(x W^T + bias) * mul
 struct QGemmEpi {
   const bf16_t* bias = nullptr;  // [O], nullable
   ActParams act;
+  const bf16_t* mul = nullptr;   // [rows][ldy], nullable
   bool out_f32 = false;
 };
 // up to four matrices of one format and row length over the same rows in one dense launch; epi

@@ -74,6 +74,7 @@ struct GemmJob {
   float* y_f32;        // non-null: float32 output instead of bfloat16
   const bf16_t* bias;  // bf16 weights only, nullable: added to the product, then the activation
   ActParams act;
+  const bf16_t* mul;   // with bias and act: multiplies the result, rows as y's, nullable
 };
 struct GemmParams {
   int njobs;
@@ -605,7 +606,10 @@ __global__ void __launch_bounds__(gemm_threads(DQW), DQW == 4 ? 4 : 1) k_qgemm(c
               if (tok < w.ntok) {
                 const size_t orow = P.row_map != nullptr ? P.row_map[w.tok0 + tok] : (size_t)(w.tok0 + tok);
                 float r = __uint_as_float(v[j]);
-                if (kDirect) r = act_apply(J.act.kind, r + ep_bias, ep_a, ep_b);
+                if (kDirect) {
+                  r = act_apply(J.act.kind, r + ep_bias, ep_a, ep_b);
+                  if (J.mul != nullptr) r *= bf2f(__ldg(J.mul + orow * J.ldy + fo));
+                }
                 if (J.y_f32 != nullptr) J.y_f32[orow * J.ldy + fo] = r;
                 else J.y[orow * J.ldy + fo] = f2bf(r);
               }
@@ -655,7 +659,10 @@ __global__ void __launch_bounds__(gemm_threads(DQW), DQW == 4 ? 4 : 1) k_qgemm(c
               for (int e = 0; e < 4; ++e)
                 if (feat + e < J.O) {
                   float r = r4[e];
-                  if (kDirect) r = act_apply(J.act.kind, r + (J.bias != nullptr ? bf2f(J.bias[feat + e]) : 0.f), ep_a, ep_b);
+                  if (kDirect) {
+                    r = act_apply(J.act.kind, r + (J.bias != nullptr ? bf2f(J.bias[feat + e]) : 0.f), ep_a, ep_b);
+                    if (J.mul != nullptr) r *= bf2f(J.mul[orow * J.ldy + feat + e]);
+                  }
                   if (J.y_f32 != nullptr) J.y_f32[orow * J.ldy + feat + e] = r;
                   else J.y[orow * J.ldy + feat + e] = f2bf(r);
                 }
@@ -849,6 +856,7 @@ int f_qgemm_multi(orn_ctx* ctx, cudaStream_t s, const orn_linear* const* Ls, voi
     J.y_f32 = f32 ? reinterpret_cast<float*>(ys[j]) : nullptr;
     J.bias = epi != nullptr ? epi[j].bias : nullptr;
     J.act = epi != nullptr ? epi[j].act : ActParams();
+    J.mul = epi != nullptr ? epi[j].mul : nullptr;
     P.f_tiles += (Ls[j]->O + BM - 1) / BM;
   }
   P.K = L->K; P.KB = (L->K + BK - 1) / BK; P.rows = rows; P.err = ctx->dev_err;

@@ -1647,7 +1647,7 @@ extern const orn_arch kArchQwen35 = {
 
 // The "architecture" of a config.json names its entry; the reference's own files have none and mean Qwen3.5-MoE.
 const orn_arch* orn_arch_of_config(const orna::JVal& cfg) {
-  static const orn_arch* const all[] = {&kArchQwen35, &kArchPeratar};
+  static const orn_arch* const all[] = {&kArchQwen35, &kArchPeratar, &kArchDokulorn};
   const orna::JVal* a = cfg.get("architecture");
   if (a == nullptr || a->type != orna::JVal::Str) return &kArchQwen35;
   for (const orn_arch* e : all)

@@ -13,7 +13,7 @@ namespace ornm {
 
 
 constexpr int kMaxRows = 4;   // widest window a forward call takes
-constexpr int kRing = 5;      // state buffers per gated-delta layer (window <= 4)
+constexpr int kRing = 5;      // state buffers per recurrent layer (window <= 4)
 
 struct Moe {
   orn_linear *gate = nullptr, *sw_gate = nullptr, *sw_up = nullptr, *sw_down = nullptr;
@@ -114,9 +114,9 @@ struct orn_model {
 struct orn_cache {
   orn_model* m = nullptr;
   std::vector<void*> latent;         // per layer (latent attention): [max_ctx][row], shared by layers that read another's
-  std::vector<bf16_t*> kc, vc;       // per layer (attention layers)
+  std::vector<bf16_t*> kc, vc;       // per layer (attention layers; float32 models keep float32 rows here)
   std::vector<bf16_t*> conv;         // per layer (gdn): [S + kMaxRows, D]
-  std::vector<float*> ring;          // per layer (gdn): [kRing][Hv,128,128]
+  std::vector<float*> ring;          // per layer (recurrent state): kRing states ([Hv,128,128]; decayed: [heads][dim][vdim])
   bf16_t** conv_table = nullptr;     // device array of the conv buffers
   int n_gdn = 0;
   bf16_t *mtp_kc = nullptr, *mtp_vc = nullptr;
