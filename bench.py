@@ -876,29 +876,32 @@ def peratar_trunk_bytes(cfg, label):
     return rows * K * 2.0
 
 
-def peratar(args):
-    """Prefill and decode throughput of the Peratar decoder (random weights, whole public calls and device
-    time), its kernels against the measured peaks, and the trunk of equal size under the same clock."""
-    pkg = load_pkg()
-    ctx = pkg.Context(int(os.environ.get("LOCAL_RANK", "0")))
-    rng = np.random.default_rng(SEED)
-    hbm, which = peaks()
-    try:
-        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
-            tf = json.load(f)["bf16_tflops"]
-    except (OSError, KeyError, ValueError):
-        tf = 1590.0
-    prompts, contexts, new = (512, 4096, 8192), (128, 8192), args.gen_tokens
-    max_ctx = max(prompts) + new + 64
-    ids = rng.integers(0, PERATAR_VOCAB, max(prompts)).astype(np.uint32)
-    sampler = ClockSampler(ctx.device)
-    sampler.start()
-    launches0 = ctx.launches()
+class DecoderBench:
+    """What the decoder workloads share: random ids, prompts and contexts, the clock record, the measurement of one model."""
 
-    def measure(model, token_bytes, z, cfg):
+    def __init__(self, args):
+        self.args = args
+        self.pkg = load_pkg()
+        self.ctx = self.pkg.Context(int(os.environ.get("LOCAL_RANK", "0")))
+        self.hbm, self.which = peaks()
+        try:
+            with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+                self.tf = json.load(f)["bf16_tflops"]
+        except (OSError, KeyError, ValueError):
+            self.tf = 1590.0
+        self.prompts, self.contexts, self.new = (512, 4096, 8192), (128, 8192), args.gen_tokens
+        self.max_ctx = max(self.prompts) + self.new + 64
+        self.ids = np.random.default_rng(SEED).integers(0, PERATAR_VOCAB, max(self.prompts)).astype(np.uint32)
+        self.sampler = ClockSampler(self.ctx.device)
+        self.sampler.start()
+        self.launches0 = self.ctx.launches()
+
+    def measure(self, model, token_bytes, label_work):
+        """Prefill and decode rates, and every kernel's share of its roofline: label_work(label, rows, keys) -> (bytes, flops) or None."""
+        args, ctx, ids, new = self.args, self.ctx, self.ids, self.new
         cache = model.make_cache()
         out = {"bytes_per_token": token_bytes, "prefill": [], "decode": [], "kernels": []}
-        for T in prompts:
+        for T in self.prompts:
             for _ in range(args.warmup):
                 cache.reset()
                 model.prefill(cache, ids[:T], 8192)
@@ -910,57 +913,162 @@ def peratar(args):
             ms = ctx.timer_stop() / args.steps
             wall = (time.perf_counter() - t0) / args.steps
             out["prefill"].append({"tokens": T, "ms": ms, "tok_s": T / ms * 1e3, "e2e_tok_s": T / wall})
-        for C in contexts:
+        for C in self.contexts:
             for i in range(args.warmup + args.steps):
                 if i == args.warmup:
                     ms = wall = 0.0
                 cache.reset()
                 t0 = time.perf_counter()
-                pkg.generate_step(model, cache, ids[:C], new, 8192)
+                self.pkg.generate_step(model, cache, ids[:C], new, 8192)
                 if i >= args.warmup:
                     ms += model.prof().total_ms / args.steps
                     wall += (time.perf_counter() - t0) / args.steps
             out["decode"].append({"context": C, "us_per_token": ms * 1e3 / new, "tok_s": new / ms * 1e3, "e2e_tok_s": new / wall,
-                                  "weight_gbs": token_bytes / (ms / new) * 1e-6, "frac_hbm": token_bytes / (ms / new) * 1e-6 / hbm})
-        T = max(prompts)
+                                  "weight_gbs": token_bytes / (ms / new) * 1e-6, "frac_hbm": token_bytes / (ms / new) * 1e-6 / self.hbm})
+        T = max(self.prompts)
         cache.reset()
         ctx.ktime_begin()
-        pkg.generate_step(model, cache, ids[:T], 16, 8192)
+        self.pkg.generate_step(model, cache, ids[:T], 16, 8192)
         for label, (n, ms) in sorted(ctx.ktime_end().items(), key=lambda kv: -kv[1][1])[:24]:
-            work = peratar_label_work(z, cfg, label, T, T)
+            work = label_work(label, T, T)
             us = 1e3 * ms / n
             k = {"kernel": label, "launches": n, "us": us}
             if work is not None:
                 b, fl = work
                 k["bound"] = "tensor" if fl else "hbm"
-                k["frac"] = fl / us * 1e-6 / tf if fl else b / us * 1e-3 / hbm
+                k["frac"] = fl / us * 1e-6 / self.tf if fl else b / us * 1e-3 / self.hbm
             out["kernels"].append(k)
         cache.free()
         return out
 
+    def report(self, metric, mid, what, sizes):
+        new = self.new
+        emit({"metric": metric, "value": mid["tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": self.args.steps,
+              "warmup": self.args.warmup, "ms_per_step": mid["us_per_token"] * new * 1e-3, "higher_is_better": True, "scaling": "weak",
+              "vs_baseline": None, "dtype": "bf16 activations, f32 residual stream and accumulate", "data": "synthetic (random-init weights and ids)",
+              "config": {"workload": what + ", 8 layers, 128-token prompt, %d greedy tokens" % new,
+                         "l2_policy": "weights read per token exceed L2 (126 MB)"},
+              "e2e": {"value": mid["e2e_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 128 * 4, "d2h_bytes_per_step": 4 * (new + 1)},
+              "gpu_launches": self.ctx.launches() - self.launches0, "clocks": self.sampler.stop(),
+              "peaks": {"hbm_gbs": self.hbm, "bf16_tflops": self.tf, "source": self.which}, "sizes": sizes})
+        self.ctx.close()
+
+
+def measure_peratar(B, z):
+    m = B.pkg.TextModel.from_config(B.ctx, peratar_config(z), max_ctx=B.max_ctx)
+    m.init_random(SEED)
+    out = B.measure(m, m.weight_bytes() - 2 * PERATAR_VOCAB * z["width"], lambda *a: peratar_label_work(z, None, *a))
+    m.free()
+    return out
+
+
+def peratar(args):
+    """Prefill and decode throughput of the Peratar decoder (random weights, whole public calls and device
+    time), its kernels against the measured peaks, and the trunk of equal size under the same clock."""
+    B = DecoderBench(args)
     sizes = []
     for z in PERATAR_SIZES:
-        m = pkg.TextModel.from_config(ctx, peratar_config(z), max_ctx=max_ctx)
-        m.init_random(SEED)
-        row = {"width": z["width"], "heads": z["heads"], "ff": z["ff"], "layers": z["layers"],
-               "peratar": measure(m, m.weight_bytes() - 2 * PERATAR_VOCAB * z["width"], z, None)}
-        m.free()
+        row = {"width": z["width"], "heads": z["heads"], "ff": z["ff"], "layers": z["layers"], "peratar": measure_peratar(B, z)}
         if z["experts"] is not None:
-            m, cfg, per_token = trunk_of_equal_size(pkg, ctx, z, max_ctx)
-            row["qwen3_5_moe_bf16"] = measure(m, per_token, z, cfg)
+            m, cfg, per_token = trunk_of_equal_size(B.pkg, B.ctx, z, B.max_ctx)
+            row["qwen3_5_moe_bf16"] = B.measure(m, per_token, lambda *a: peratar_label_work(z, cfg, *a))
             m.free()
         sizes.append(row)
-    clocks = sampler.stop()
-    mid = sizes[1]["peratar"]["decode"][0]
-    emit({"metric": "Peratar decode throughput", "value": mid["tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
-          "warmup": args.warmup, "ms_per_step": mid["us_per_token"] * new * 1e-3, "higher_is_better": True, "scaling": "weak",
-          "vs_baseline": None, "dtype": "bf16 activations, f32 residual stream and accumulate", "data": "synthetic (random-init weights and ids)",
-          "config": {"workload": "width 2048, 16 heads, latent 512 + 64, ff 8192, 8 layers, 128-token prompt, %d greedy tokens" % new,
-                     "l2_policy": "weights read per token exceed L2 (126 MB)"},
-          "e2e": {"value": mid["e2e_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 128 * 4, "d2h_bytes_per_step": 4 * (new + 1)},
-          "gpu_launches": ctx.launches() - launches0, "clocks": clocks, "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": which},
-          "sizes": sizes})
-    ctx.close()
+    B.report("Peratar decode throughput", sizes[1]["peratar"]["decode"][0], "width 2048, 16 heads, latent 512 + 64, ff 8192", sizes)
+
+
+# ---- the Dokulorn decoder beside the Peratar decoder of equal size and the trunk's gated-delta layers
+def dokulorn_config(z):
+    """Heads of 128 everywhere; every fourth layer has both mixers, the others a decayed state alone.  A gated
+    feed-forward of 2/3 the width holds as much as the other decoder's plain one."""
+    H, ff = z["heads"], -(-z["ff"] * 2 // 3 // 64) * 64
+    decay = [1.0 - 2.0 ** (-4 - 6 * h / H) for h in range(H)]
+    ls = []
+    for i in range(z["layers"]):
+        state = {"heads": H, "dim": 128, "vdim": 128, "decay": decay}
+        if i % 4 == 2:
+            left = {"heads": H, "kv_heads": H // 4, "dim": 128, "vdim": 128, "rot": {"base": 1e4, "dims": 64}, "scale": 0.1, "softcap": 30.0}
+            ls.append({"type": "parallel", "mixer": {"left": left, "right": state}, "mlp": {"kind": "dense", "ff": ff}})
+        else:
+            ls.append({"type": "retention", "mixer": dict(state, rot={"base": 1e4, "dims": 128}), "mlp": {"kind": "dense", "ff": ff}})
+    return {"architecture": "Dokulorn", "width": z["width"], "vocab": PERATAR_VOCAB, "norm": {"eps": 1e-6}, "embedding": {"scale": z["width"] ** 0.5},
+            "postln_alpha": 2.0, "layers": ls}
+
+
+def dokulorn_label_work(z, label, T, ctx_len):
+    """(bytes, flops) a launch with this label has to move or compute."""
+    H, w, d = z["heads"], z["width"], 128
+    G, pairs, state = H // 4, T * (T + 1) / 2, 4.0 * H * d * d
+    rows2, chunks = 2.0 * T * H * d, -(-T // 256)  # bytes of a bf16 projection of all heads; kept states
+    if label.startswith("decode_dense"):
+        O, K = (int(v) for v in label.split()[-1].split("x"))
+        return O * K * 2.0, 0
+    if label == "decayed_window":
+        return 2 * state, 0
+    if label.startswith("grouped_window"):
+        return ctx_len * 2 * G * d * 2.0 + (2 * state if "decayed" in label else 0), 0
+    if label == "grouped_flash":
+        return 0, 2.0 * H * pairs * 2 * d
+    if label == "decayed_fold":
+        return 2 * rows2 + chunks * state, 0
+    if label == "decayed_carry":
+        return 2 * chunks * state, 0
+    if label == "decayed_rows":
+        return 3 * rows2 + 2 * rows2 + chunks * state, 0
+    if label == "group_gate_rows":
+        return (4 + 2 + 2) * T * H * d, 0
+    if label.startswith("post_norm_rows"):
+        return T * w * (3 * 4 + 2 + (4 if "pair" in label else 0)), 0
+    if label.startswith("k_qgemm kind=3"):
+        f = dict(x.split("=") for x in label.split() if "=" in x)
+        O, K, rows = int(f["O"].rstrip("+")), int(f["K"]), int(f["rows"])
+        if "+" in f["O"]:  # four projections of one input: all heads, or (3 : 1 launches over) H + G + G + H heads; the mean of both kinds
+            n = z["layers"]
+            par = n // 4
+            O = ((n - par) * 4 * H * d + par * (4 * H * d + 2 * (H + G) * d)) / (n + par)
+        return 0, 2.0 * O * K * rows
+    return None
+
+
+def gated_delta_label_work(cfg, label, T, ctx_len):
+    """The trunk's recurrent layers and its attention."""
+    Hv, Hk, d = cfg.gdn_v_heads, cfg.gdn_k_heads, cfg.gdn_head_dim
+    state, v2, k2 = 4.0 * Hv * d * d, 2.0 * T * Hv * d, 2.0 * T * Hk * d
+    if label == "k_gdn":
+        return 2 * state, 0
+    if label == "gdn_chunk_prep":  # q and k in, five operand tiles per 64 tokens and head out
+        return 2 * k2 + T / 64 * Hv * (3 * 64 * d + 2 * 64 * 64) * 2.0, 0
+    if label == "gdn_chunk_scan":
+        return T / 64 * Hv * (3 * 64 * d + 2 * 64 * 64) * 2.0 + 2 * v2 + 2 * state, 0
+    if label == "flash_prefill":
+        return 0, 2.0 * cfg.n_heads * T * (T + 1) / 2 * 2 * cfg.head_dim
+    if label in ("k_attn", "k_attn_split"):
+        return ctx_len * 2 * cfg.n_kv_heads * cfg.head_dim * 2.0, 0
+    return None
+
+
+def dokulorn(args):
+    """Prefill and decode throughput of the Dokulorn decoder (random weights), its kernels against the measured peaks;
+    beside it the Peratar decoder of equal size and the trunk's gated-delta layers under the same clock."""
+    B = DecoderBench(args)
+    sizes = []
+    for z in PERATAR_SIZES:
+        m = B.pkg.TextModel.from_config(B.ctx, dokulorn_config(z), max_ctx=B.max_ctx)
+        m.init_random(SEED)
+        row = {"width": z["width"], "heads": z["heads"], "layers": z["layers"],
+               "dokulorn": B.measure(m, m.weight_bytes(), lambda *a: dokulorn_label_work(z, *a))}
+        m.free()
+        row["peratar"] = measure_peratar(B, z)
+        if z["width"] == 2048:
+            E, k, inter, shared = z["experts"]
+            cfg = B.pkg.qwen35_config(max_ctx=B.max_ctx, n_layers=z["layers"], n_experts=E, top_k=k, expert_inter=inter, shared_inter=shared,
+                                      vocab=PERATAR_VOCAB)
+            m = B.pkg.TextModel(B.ctx, cfg)
+            m.init_random(SEED)
+            row["qwen3_5_moe_quantised"] = B.measure(m, m.weight_bytes(), lambda *a: gated_delta_label_work(cfg, *a))
+            m.free()
+        sizes.append(row)
+    B.report("Dokulorn decode throughput", sizes[1]["dokulorn"]["decode"][0], "width 2048, 16 heads of 128, gated ff 5504", sizes)
 
 
 def ep_layer(args):
@@ -1108,9 +1216,10 @@ def main():
     ap.add_argument("--n-layers", type=int, default=40, help="fewer layers at the full layer sizes (profiling runs)")
     ap.add_argument("--long-prefill", action="store_true", help="run the 6621-token prefill leg at any layer count")
     ap.add_argument("--ep-decode", action="store_true", help="run the batched expert-parallel decode leg at any layer count")
-    ap.add_argument("--workload", default="decode", choices=["decode", "ep-layer", "peratar"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "ep-layer", "peratar", "dokulorn"],
                     help="decode: the MTP depth-1 decode loop (the headline); ep-layer: one expert-parallel MoE layer; "
-                         "peratar: prefill and decode of the Peratar decoder beside the trunk of equal size (1 GPU)")
+                         "peratar: prefill and decode of the Peratar decoder beside the trunk of equal size (1 GPU); "
+                         "dokulorn: the same of the Dokulorn decoder beside the Peratar decoder and the trunk (1 GPU)")
     args = ap.parse_args()
     global GEN_TOKENS, PROMPT_LEN
     GEN_TOKENS, PROMPT_LEN = args.gen_tokens, args.prompt_len
@@ -1120,6 +1229,8 @@ def main():
         ep_layer(args)
     elif args.workload == "peratar":
         peratar(args)
+    elif args.workload == "dokulorn":
+        dokulorn(args)
     else:
         ours(args)
 
