@@ -41,4 +41,21 @@ ORN_D float act_apply(int kind, float z, float a, float b) {
   if (kind == ACT_GELU_TANH) return gelu_tanh_f32(z);
   return z;
 }
+// N values at once: the kind is looked at once, and an unrolled caller holds every activation's code
+// N times in a row instead of all of them between any two values
+template <int N> ORN_D void act_apply_n(int kind, float* z, float a, float b) {
+#define ORN_ACT_CASE(K)                                       \
+  case K:                                                     \
+    _Pragma("unroll") for (int i = 0; i < N; ++i) z[i] = act_apply(K, z[i], a, b); \
+    break
+  switch (kind) {
+    ORN_ACT_CASE(ACT_XIELU);
+    ORN_ACT_CASE(ACT_SOFTCAP);
+    ORN_ACT_CASE(ACT_SILU);
+    ORN_ACT_CASE(ACT_SIGMOID);
+    ORN_ACT_CASE(ACT_GELU_TANH);
+    default: break;
+  }
+#undef ORN_ACT_CASE
+}
 #endif

@@ -600,20 +600,28 @@ __global__ void __launch_bounds__(gemm_threads(DQW), DQW == 4 ? 4 : 1) k_qgemm(c
               if (tok < w.ntok) part[(size_t)tok * BM + q * 32 + lane] = __uint_as_float(v[j]);
             }
           } else if (fo < J.O) {
+            float r[16];
 #pragma unroll
-            for (int j = 0; j < 16; ++j) {
-              const int tok = t * P.BN + c0 + j;
-              if (tok < w.ntok) {
-                const size_t orow = P.row_map != nullptr ? P.row_map[w.tok0 + tok] : (size_t)(w.tok0 + tok);
-                float r = __uint_as_float(v[j]);
-                if (kDirect) {
-                  r = act_apply(J.act.kind, r + ep_bias, ep_a, ep_b);
-                  if (J.mul != nullptr) r *= bf2f(__ldg(J.mul + orow * J.ldy + fo));
-                }
-                if (J.y_f32 != nullptr) J.y_f32[orow * J.ldy + fo] = r;
-                else J.y[orow * J.ldy + fo] = f2bf(r);
+            for (int j = 0; j < 16; ++j) r[j] = kDirect ? __uint_as_float(v[j]) + ep_bias : __uint_as_float(v[j]);
+            const int tok0 = t * P.BN + c0, n = w.ntok - tok0;  // n > 0
+            if (kDirect) {
+              act_apply_n<16>(J.act.kind, r, ep_a, ep_b);
+              if (J.mul != nullptr) {  // dense products only: rows in order
+                const bf16_t* mp = J.mul + (size_t)(w.tok0 + tok0) * J.ldy + fo;
+                bf16_t f[16];
+#pragma unroll
+                for (int j = 0; j < 16; ++j) f[j] = j < n ? __ldg(mp + (size_t)j * J.ldy) : (bf16_t)0;
+#pragma unroll
+                for (int j = 0; j < 16; ++j) r[j] *= bf2f(f[j]);
               }
             }
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+              if (j < n) {
+                const size_t orow = P.row_map != nullptr ? P.row_map[w.tok0 + tok0 + j] : (size_t)(w.tok0 + tok0 + j);
+                if (J.y_f32 != nullptr) J.y_f32[orow * J.ldy + fo] = r[j];
+                else J.y[orow * J.ldy + fo] = f2bf(r[j]);
+              }
           }
         }
       }
@@ -654,13 +662,18 @@ __global__ void __launch_bounds__(gemm_threads(DQW), DQW == 4 ? 4 : 1) k_qgemm(c
               const int tok = i / (BM / 4), f = 4 * (i - tok * (BM / 4));
               const int feat = w.ft * BM + f;
               const size_t orow = (size_t)(w.tok0 + tok);
-              const float r4[4] = {acc[u].x, acc[u].y, acc[u].z, acc[u].w};
+              float r4[4] = {acc[u].x, acc[u].y, acc[u].z, acc[u].w};
+              if (kDirect) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                  if (J.bias != nullptr && feat + e < J.O) r4[e] += bf2f(J.bias[feat + e]);
+                act_apply_n<4>(J.act.kind, r4, ep_a, ep_b);
+              }
 #pragma unroll
               for (int e = 0; e < 4; ++e)
                 if (feat + e < J.O) {
                   float r = r4[e];
                   if (kDirect) {
-                    r = act_apply(J.act.kind, r + (J.bias != nullptr ? bf2f(J.bias[feat + e]) : 0.f), ep_a, ep_b);
                     if (J.mul != nullptr) r *= bf2f(J.mul[orow * J.ldy + feat + e]);
                   }
                   if (J.y_f32 != nullptr) J.y_f32[orow * J.ldy + feat + e] = r;
