@@ -58,6 +58,7 @@ constexpr int gemm_threads(int dqw) { return 64 + 32 * dqw; }
 constexpr uint32_t kAccColsMax = 384;   // accumulator columns of an item: the rest of tensor memory holds weight tiles
 constexpr uint32_t kWCols = BK / 2;     // tensor-memory columns of one dequantised 128 x 64 tile (two bf16 per column)
 constexpr int kSplitMaxRows = 512;                      // dense products up to this many rows may split K
+constexpr int kSplitMaxRowsEpi = 128;                   // ... with an epilogue: its callers' rows may differ in rounding, and the partials of more rows cost more than they save
 constexpr size_t kSplitPartialBytes = (size_t)64 << 20;  // f32 partials of one launch
 constexpr size_t kSplitTiles = 4096;                     // arrival counters
 constexpr uint32_t kWTileBytes = BM * BK * 2;
@@ -905,7 +906,7 @@ int f_qgemm_multi(orn_ctx* ctx, cudaStream_t s, const orn_linear* const* Ls, voi
   // (O, K) only, never on the row count, so that a row's bits do not depend on how many rows share
   // the launch.
   P.splits = 1; P.partial = nullptr; P.arrivals = nullptr;
-  if (grp == nullptr && rows <= kSplitMaxRows && P.KB >= 8) {
+  if (grp == nullptr && rows <= (epi != nullptr ? kSplitMaxRowsEpi : kSplitMaxRows) && P.KB >= 8) {
     const int tiles = P.f_tiles * ((rows + P.NT * BN - 1) / (P.NT * BN));
     // one round of items over the SMs, two CTAs on each where the tiles alone would leave SMs idle
     // (97 tiles of an input projection: three splits instead of none)
