@@ -97,6 +97,38 @@ ORN_D void group_gate_row(const GroupGate& G, int m, TA* out, float* stash, floa
     for (int e = 0; e < 4; ++e)
       if (d + e < G.group) out[at + e] = to_act<TA>(v[e]);
   };
+  if (vec && G.group <= 128) {  // four groups at a time, all requested before the first is used
+    constexpr int kAhead = 4;
+    const int step = (THREADS / 32) * G.group, d = 4 * lane;
+    for (int g0 = warp * G.group; g0 < G.n; g0 += kAhead * step) {
+      float v[kAhead][4], z[kAhead][4], w[kAhead][4];
+#pragma unroll
+      for (int k = 0; k < kAhead; ++k) {
+        const int at = g0 + k * step, n = at < G.n ? G.group : 0;
+        load_row4(o + at, d, n, true, v[k]);
+        load_row4(gate + at, d, n, true, z[k]);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) w[k][e] = 1.f;
+        if (G.w != nullptr) load_bf4(G.w + at, d, n, w[k]);
+      }
+#pragma unroll
+      for (int k = 0; k < kAhead; ++k) {
+        const int at = g0 + k * step;
+        if (at >= G.n) break;  // warp-uniform
+        float sq = 0.f;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sq = fmaf(v[k][e], v[k][e], sq);
+        const float rstd = 1.0f / sqrtf(warp_sum(sq) * inv + G.eps);
+        if (d < G.group) {
+          act_apply_n<4>(G.act, z[k], 0.f, 0.f);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) v[k][e] = v[k][e] * rstd * w[k][e] * z[k][e];
+          store_act4(out + at + d, v[k]);
+        }
+      }
+    }
+    return;
+  }
   if (group_gate_warp(G)) {
     for (int g0 = warp * G.group; g0 < G.n; g0 += (THREADS / 32) * G.group) {
       float v[kGgRegs][4], z[kGgRegs][4], sq = 0.f;

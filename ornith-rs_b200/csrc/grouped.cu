@@ -102,7 +102,7 @@ __global__ void __launch_bounds__(kGpThreads) grouped_plain_kernel(GroupedDims D
 }
 
 // ------------------------------------------------------------------ decode windows
-constexpr int kGwWarps = 8, kGwThreads = 32 * kGwWarps, kGwKeys = 64, kGwMaxSplits = 64, kGwMaxRows = 4;
+constexpr int kGwWarps = 8, kGwThreads = 32 * kGwWarps, kGwKeys = 64, kGwMaxSplits = 64, kGwMaxRows = 4, kGwTeams = 8;
 static_assert(kGwThreads == kDwThreads, "attention and decayed state share a launch");
 struct WindowArgs {
   GroupedArgs a;
@@ -179,21 +179,33 @@ ORN_D void grouped_window_cta(const GroupedDims& D, const WindowArgs& W, uint8_t
   pdl_wait();
   pdl_trigger();
   __syncthreads();
+  // the rows as they come wait in the second tile buffer, which is not in use yet: one request each
+  uint8_t* raw = smem + L.tiles + L.stage;
+  auto fetch = [&](int slot, const bf16_t* src) {
+    for (int c = lane; c < dp; c += 32) *reinterpret_cast<uint4*>(raw + slot * L.rowB + 16 * c) = __ldcg(reinterpret_cast<const uint4*>(src) + c);
+  };
   auto norm_of = [&](const bf16_t* src) {
     if (!D.unit_qk) return 1.0f;
     float sq = 0.f;
-    for (int d = lane; d < D.dim; d += 32) { const float v = bf2f(__ldcg(src + d)); sq = fmaf(v, v, sq); }
+    for (int d = lane; d < D.dim; d += 32) { const float v = bf2f(src[d]); sq = fmaf(v, v, sq); }
     return 1.0f / sqrtf(warp_sum(sq) / (float)D.dim + D.eps);  // turning keeps the length
   };
+  for (int r = warp; r < 16 && r0 + r < rows; r += kGwWarps) {
+    const int t = (r0 + r) / rep, h = j * rep + r0 + r - t * rep;
+    fetch(r, reinterpret_cast<const bf16_t*>(A.q) + (size_t)t * A.ldq + (size_t)h * D.dim);
+  }
+  for (int t = kGwWarps - 1 - warp; t < T; t += kGwWarps)
+    if (p0 + t >= k0 && p0 + t < k1) fetch(16 + t, reinterpret_cast<const bf16_t*>(A.k) + (size_t)t * A.ldk + (size_t)j * D.dim);
+  __syncwarp();  // a warp reads what it fetched
   for (int r = warp; r < 16; r += kGwWarps) {
     bf16_t* dst = reinterpret_cast<bf16_t*>(smem + L.q + r * L.rowB);
     const int row = r0 + r;
     if (row < rows) {
-      const int t = row / rep, h = j * rep + row - t * rep;
-      const bf16_t* src = reinterpret_cast<const bf16_t*>(A.q) + (size_t)t * A.ldq + (size_t)h * D.dim;
+      const int t = row / rep;
+      const bf16_t* src = reinterpret_cast<const bf16_t*>(raw + r * L.rowB);
       const float rn = norm_of(src);
       for (int d = lane; d < KD; d += 32)
-        dst[d] = d < D.dim ? f2bf(rn * rotated_half(d, half, s_cs + t * half, [&](int e) { return bf2f(__ldcg(src + e)); })) : (bf16_t)0;
+        dst[d] = d < D.dim ? f2bf(rn * rotated_half(d, half, s_cs + t * half, [&](int e) { return bf2f(src[e]); })) : (bf16_t)0;
     } else {
       for (int d = lane; d < KD; d += 32) dst[d] = 0;
     }
@@ -201,11 +213,11 @@ ORN_D void grouped_window_cta(const GroupedDims& D, const WindowArgs& W, uint8_t
   for (int t = kGwWarps - 1 - warp; t < T; t += kGwWarps) {
     const int key = p0 + t;
     if (key < k0 || key >= k1) continue;  // warp-uniform
-    const bf16_t* src = reinterpret_cast<const bf16_t*>(A.k) + (size_t)t * A.ldk + (size_t)j * D.dim;
+    const bf16_t* src = reinterpret_cast<const bf16_t*>(raw + (16 + t) * L.rowB);
     bf16_t *nk = reinterpret_cast<bf16_t*>(smem + L.nk) + t * D.dim, *nv = reinterpret_cast<bf16_t*>(smem + L.nv) + t * D.vdim;
     const float rn = norm_of(src);
     for (int d = lane; d < D.dim; d += 32) {
-      const bf16_t v = f2bf(rn * rotated_half(d, half, s_cs + t * half, [&](int e) { return bf2f(__ldcg(src + e)); }));
+      const bf16_t v = f2bf(rn * rotated_half(d, half, s_cs + t * half, [&](int e) { return bf2f(src[e]); }));
       nk[d] = v;
       if (r0 == 0) kc[(size_t)key * A.ldkc + d] = v;
     }
@@ -372,12 +384,36 @@ ORN_D void grouped_window_cta(const GroupedDims& D, const WindowArgs& W, uint8_t
   }
   __syncthreads();
   const float* ps = W.partial + (size_t)jm * W.splits * 16 * D.vdim;
-  for (int i = threadIdx.x; i < nr * D.vdim; i += kGwThreads) {
-    const int r = i / D.vdim;
-    float a = 0.f;
+  // four columns per thread; where that leaves threads over, they share the ranges
+  const int units = nr * D.vdim / 4, teams = max(1, min(kGwTeams, kGwThreads / units));
+  float4* s_acc = reinterpret_cast<float4*>(smem + L.tiles);
+  for (int u0 = 0; u0 < units; u0 += kGwThreads) {
+    const int team = teams > 1 ? threadIdx.x / units : 0, u = teams > 1 ? threadIdx.x - team * units : u0 + threadIdx.x;
+    const bool on = u < units && team < teams;
+    const int r = 4 * u / D.vdim;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (on) {
 #pragma unroll 8
-    for (int sp = 0; sp < used; ++sp) a = fmaf(s_w[r * kGwMaxSplits + sp], __ldcg(ps + (size_t)sp * 16 * D.vdim + i), a);
-    put(r0 + r, i - r * D.vdim, a * s_inv[r]);
+      for (int sp = team; sp < used; sp += teams) {
+        const float w = s_w[r * kGwMaxSplits + sp];
+        const float4 v = __ldcg(reinterpret_cast<const float4*>(ps + (size_t)sp * 16 * D.vdim) + u);
+        a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y); a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
+      }
+    }
+    if (teams > 1) {  // one round: the same for every thread
+      if (on) s_acc[team * units + u] = a;
+      __syncthreads();
+      if (on && team == 0)
+        for (int k = 1; k < teams; ++k) {
+          const float4 v = s_acc[k * units + u];
+          a.x += v.x; a.y += v.y; a.z += v.z; a.w += v.w;
+        }
+    }
+    if (on && team == 0) {
+      const int col = 4 * u - r * D.vdim;
+      const float inv = s_inv[r];
+      put(r0 + r, col, a.x * inv); put(r0 + r, col + 1, a.y * inv); put(r0 + r, col + 2, a.z * inv); put(r0 + r, col + 3, a.w * inv);
+    }
   }
   if (threadIdx.x == 0) W.arrivals[jm] = 0;  // ready for the next launch
 }
