@@ -80,6 +80,14 @@ ORN_D void load_row4(const bf16_t* p, int d, int n, bool vec, float* v) {
   for (int e = 0; e < 4; ++e) v[e] = d + e < n ? bf2f(__ldcg(p + d + e)) : 0.f;
 }
 
+// the gate of a mixer's heads: sigmoid(z) or, for ACT_SILU, z sigmoid(z)
+ORN_D float head_gate(int act, float z) {
+  const float s = sigmoid_f32(z);
+  return act == ACT_SILU ? z * s : s;
+}
+// An activation as a call: decode kernels run once through their code, which should be short.
+__device__ __noinline__ float act_apply_call(int kind, float z, float a, float b) { return act_apply(kind, z, a, b); }
+
 // Row m of a mixer's heads under their group norm and gate.  A warp per group while a group fits its
 // registers, the whole block otherwise.  stash: group_gate_stash() floats; red: as block_sum.
 constexpr int kGgRegs = 4;  // groups of up to kGgRegs * 128 entries stay in a warp's registers
@@ -120,9 +128,8 @@ ORN_D void group_gate_row(const GroupGate& G, int m, TA* out, float* stash, floa
         for (int e = 0; e < 4; ++e) sq = fmaf(v[k][e], v[k][e], sq);
         const float rstd = 1.0f / sqrtf(warp_sum(sq) * inv + G.eps);
         if (d < G.group) {
-          act_apply_n<4>(G.act, z[k], 0.f, 0.f);
 #pragma unroll
-          for (int e = 0; e < 4; ++e) v[k][e] = v[k][e] * rstd * w[k][e] * z[k][e];
+          for (int e = 0; e < 4; ++e) v[k][e] = v[k][e] * rstd * w[k][e] * head_gate(G.act, z[k][e]);
           store_act4(out + at + d, v[k]);
         }
       }
@@ -150,7 +157,7 @@ ORN_D void group_gate_row(const GroupGate& G, int m, TA* out, float* stash, floa
           float w[4] = {1.f, 1.f, 1.f, 1.f};
           if (G.w != nullptr) load_bf4(G.w + g0, d, G.group, w);
 #pragma unroll
-          for (int e = 0; e < 4; ++e) v[it][e] = v[it][e] * rstd * w[e] * act_apply(G.act, z[it][e], 0.f, 0.f);
+          for (int e = 0; e < 4; ++e) v[it][e] = v[it][e] * rstd * w[e] * head_gate(G.act, z[it][e]);
           put(g0 + d, d, v[it]);
         }
       }
@@ -167,7 +174,7 @@ ORN_D void group_gate_row(const GroupGate& G, int m, TA* out, float* stash, floa
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         sq = fmaf(v[e], v[e], sq);
-        if (d + e < G.group) stash[d + e] = v[e] * w[e] * act_apply(G.act, z[e], 0.f, 0.f);
+        if (d + e < G.group) stash[d + e] = v[e] * w[e] * head_gate(G.act, z[e]);
       }
     }
     const float rstd = 1.0f / sqrtf(block_sum<THREADS>(sq, red) * inv + G.eps);
@@ -423,28 +430,30 @@ struct DecParams {
   DecJobDev job[kDecJobs];
 };
 
-// M rows staged as bf16 [M][Kp]: heads under their norm and gate, or the residual normed after its sum.
+// M rows staged as bf16 [M][Kp]: plain entries, then heads under their norm and gate.
+template <int M>
+ORN_D void decode_prologue_gated(const DecParams& P, bf16_t* s_x, float* f, float* red) {
+  const DecodePrologue& p = P.p;
+  const int Kp = P.Kp, Kr = (p.K + 7) & ~7;
+  for (int i = threadIdx.x; i < M * (Kr / 8); i += kDecThreads) {
+    const int m = i / (Kr / 8), c = i - m * (Kr / 8);
+    *reinterpret_cast<uint4*>(s_x + (size_t)m * Kp + 8 * c) = __ldcg(reinterpret_cast<const uint4*>(p.rows + (size_t)m * p.ldx) + c);
+  }
+#pragma unroll 1
+  for (int m = 0; m < M; ++m) {
+    bf16_t* xs = s_x + (size_t)m * Kp + Kr;
+    group_gate_row<kDecThreads, bf16_t>(p.gg, m, xs, f, red);
+    if ((int)threadIdx.x < Kp - Kr - p.gg.n) xs[p.gg.n + threadIdx.x] = 0;
+    if (!group_gate_warp(p.gg)) __syncthreads();  // the stash is reused by the next row
+  }
+  __syncthreads();
+}
+// M rows staged as bf16 [M][Kp]: the residual normed after its sum.
 template <int M>
 ORN_D void decode_prologue_post(const DecParams& P, bf16_t* s_x, float* f, float* red) {
   const DecodePrologue& p = P.p;
   const int Kp = P.Kp, K = p.K;
   const bool lead = blockIdx.x == 0;
-  if (p.mode == DRO_GATED) {
-    const int Kr = (K + 7) & ~7;
-    for (int i = threadIdx.x; i < M * (Kr / 8); i += kDecThreads) {
-      const int m = i / (Kr / 8), c = i - m * (Kr / 8);
-      *reinterpret_cast<uint4*>(s_x + (size_t)m * Kp + 8 * c) = __ldcg(reinterpret_cast<const uint4*>(p.rows + (size_t)m * p.ldx) + c);
-    }
-#pragma unroll 1
-    for (int m = 0; m < M; ++m) {
-      bf16_t* xs = s_x + (size_t)m * Kp + Kr;
-      group_gate_row<kDecThreads, bf16_t>(p.gg, m, xs, f, red);
-      if ((int)threadIdx.x < Kp - Kr - p.gg.n) xs[p.gg.n + threadIdx.x] = 0;
-      if (!group_gate_warp(p.gg)) __syncthreads();  // the stash is reused by the next row
-    }
-    __syncthreads();
-    return;
-  }
   const PostNormStep& Q = p.pn;
   const float inv = 1.0f / (float)K;
   const bool pair = Q.y2 != nullptr;
@@ -722,8 +731,9 @@ ORN_D void decode_prologue(const DecParams& P, bf16_t* s_x, float* s_f, float* r
 }
 
 // A warp takes R consecutive rows of one matrix: 32 lanes x 16 bytes per step and row, U steps in flight.
-// POST: the prologues of decode_prologue_post, the others otherwise.
-template <int M, int R, int U, bool POST>
+// One instance per family of prologues: an instance holds the code of its own only.
+enum { PF_STREAM = 0, PF_POSTNORM = 1, PF_GATED = 2 };
+template <int M, int R, int U, int PF>
 __global__ void __launch_bounds__(kDecThreads) decode_dense_kernel(const __grid_constant__ DecParams P) {
   extern __shared__ __align__(16) uint8_t s_raw[];
   __shared__ float red[33], s_act[kDecJobs][2];
@@ -759,7 +769,8 @@ __global__ void __launch_bounds__(kDecThreads) decode_dense_kernel(const __grid_
   if (threadIdx.x < P.njobs) act_prepare(P.job[threadIdx.x].act, s_act[threadIdx.x][0], s_act[threadIdx.x][1]);
   pdl_wait();
   pdl_trigger();
-  if (POST) decode_prologue_post<M>(P, s_x, s_f, red);
+  if (PF == PF_POSTNORM) decode_prologue_post<M>(P, s_x, s_f, red);
+  else if (PF == PF_GATED) decode_prologue_gated<M>(P, s_x, s_f, red);
   else decode_prologue<M>(P, s_x, s_f, red);
   for (; task < P.tasks; task += stride) {
     float acc[R][M];
@@ -807,7 +818,7 @@ __global__ void __launch_bounds__(kDecThreads) decode_dense_kernel(const __grid_
 #pragma unroll
       for (int m = 0; m < M; ++m)
         if (lane == m) {
-          const float v = act_apply(J.act.kind, acc[0][m], s_act[jj][0], s_act[jj][1]) * acc[R - 1][m];
+          const float v = act_apply_call(J.act.kind, acc[0][m], s_act[jj][0], s_act[jj][1]) * acc[R - 1][m];
           if (J.out_f32) reinterpret_cast<float*>(J.y)[(size_t)m * J.ldy + oo] = v;
           else reinterpret_cast<bf16_t*>(J.y)[(size_t)m * J.ldy + oo] = f2bf(v);
         }
@@ -822,7 +833,8 @@ __global__ void __launch_bounds__(kDecThreads) decode_dense_kernel(const __grid_
         if (lane == r * M + m) { mine = acc[r][m]; mr = r; mm = m; }
     if (lane < R * M && oo + mr < J.O) {
       const int o = oo + mr;
-      const float v = act_apply(J.act.kind, mine + (J.bias != nullptr ? bf2f(J.bias[o]) : 0.f), s_act[jj][0], s_act[jj][1]);
+      float v = mine + (J.bias != nullptr ? bf2f(J.bias[o]) : 0.f);
+      if (J.act.kind != ACT_NONE) v = act_apply_call(J.act.kind, v, s_act[jj][0], s_act[jj][1]);
       if (J.out_f32) reinterpret_cast<float*>(J.y)[(size_t)mm * J.ldy + o] = v;
       else reinterpret_cast<bf16_t*>(J.y)[(size_t)mm * J.ldy + o] = f2bf(v);
     }
@@ -836,13 +848,13 @@ size_t decode_smem(const DecodePrologue& p, int M) {
   return (((size_t)M * Kp * 2 + 15) & ~(size_t)15) + floats * 4;
 }
 
-template <int M, int R, int U, bool POST>
+template <int M, int R, int U, int PF>
 int launch_decode(orn_ctx* ctx, cudaStream_t s, const DecParams& P, int grid, size_t smem, const char* label) {
   if (smem > 48 * 1024) {
-    const int rc = orn_grant_smem(ctx, reinterpret_cast<const void*>(decode_dense_kernel<M, R, U, POST>), kDecSmemMax);
+    const int rc = orn_grant_smem(ctx, reinterpret_cast<const void*>(decode_dense_kernel<M, R, U, PF>), kDecSmemMax);
     if (rc != ORN_OK) return rc;
   }
-  ORN_CHECK_CUDA(ctx, orn_launch_dependent(ctx, s, 0, decode_dense_kernel<M, R, U, POST>, dim3(grid), dim3(kDecThreads), smem, P));
+  ORN_CHECK_CUDA(ctx, orn_launch_dependent(ctx, s, 0, decode_dense_kernel<M, R, U, PF>, dim3(grid), dim3(kDecThreads), smem, P));
   return orn_launch_check(ctx, label);
 }
 
@@ -882,7 +894,7 @@ int k_rms_norm_rows(orn_ctx* ctx, cudaStream_t s, const float* x, int rows, int 
 }
 
 int k_group_gate_rows(orn_ctx* ctx, cudaStream_t s, int rows, const GroupGate& g, void* out, int ldout, bool act_f32) {
-  if (g.group < 1 || g.n % g.group) ORN_FAIL(ctx, ORN_ERR_ARG, "group gate: whole groups only");
+  if (g.group < 1 || g.n % g.group || (g.act != ACT_SILU && g.act != ACT_SIGMOID)) ORN_FAIL(ctx, ORN_ERR_ARG, "group gate: whole groups, sigmoid or SiLU");
   if (g.ldo % 8 || g.ldg % 8 || ldout % 8) ORN_FAIL(ctx, ORN_ERR_ARG, "group gate: row strides must be multiples of 8");
   const size_t smem = sizeof(float) * group_gate_stash(g);
   if (smem > kDecSmemMax) ORN_FAIL(ctx, ORN_ERR_ARG, "group gate: a group above 51200 entries");
@@ -958,7 +970,7 @@ int f_decode_dense(orn_ctx* ctx, cudaStream_t s, int M, const DecodePrologue& p,
   if (p.mode == DRO_ROWS && (p.ldx % 8 || p.ldx < P.Kp)) ORN_FAIL(ctx, ORN_ERR_ARG, "decode product: row stride");
   if (p.mode == DRO_RESIDUAL && p.r.ld != P.Kp) ORN_FAIL(ctx, ORN_ERR_ARG, "decode product: residual stride");
   if (p.mode == DRO_POSTNORM && p.pn.ld != P.Kp) ORN_FAIL(ctx, ORN_ERR_ARG, "decode product: residual stride");
-  if (p.mode == DRO_GATED && (p.gg.group < 1 || p.gg.n % p.gg.group || p.gg.ldo % 8 || p.gg.ldg % 8 || (p.K > 0 && (p.ldx % 8 || p.ldx < pad8(p.K)))))
+  if (p.mode == DRO_GATED && (p.gg.group < 1 || p.gg.n % p.gg.group || (p.gg.act != ACT_SILU && p.gg.act != ACT_SIGMOID) || p.gg.ldo % 8 || p.gg.ldg % 8 || (p.K > 0 && (p.ldx % 8 || p.ldx < pad8(p.K)))))
     ORN_FAIL(ctx, ORN_ERR_ARG, "decode product: gated rows");
   long total = 0;
   bool pairs = false;
@@ -996,14 +1008,14 @@ int f_decode_dense(orn_ctx* ctx, cudaStream_t s, int M, const DecodePrologue& p,
     std::lock_guard<std::mutex> lock(mu);
     label = pool.insert(t).first->c_str();
   }
-  const bool post = p.mode == DRO_POSTNORM || p.mode == DRO_GATED;
-#define ORN_DEC(M_)                                                                                             \
-  case M_:                                                                                                      \
-    if (post)                                                                                                   \
-      return R == 2 ? launch_decode<M_, 2, 4, true>(ctx, s, P, grid, smem, label)                               \
-                    : launch_decode<M_, 1, 8, true>(ctx, s, P, grid, smem, label);                              \
-    return R == 2 ? launch_decode<M_, 2, 4, false>(ctx, s, P, grid, smem, label)                                \
-                  : launch_decode<M_, 1, 8, false>(ctx, s, P, grid, smem, label)
+#define ORN_DEC_PF(M_, PF_)                                                       \
+  return R == 2 ? launch_decode<M_, 2, 4, PF_>(ctx, s, P, grid, smem, label)      \
+                : launch_decode<M_, 1, 8, PF_>(ctx, s, P, grid, smem, label)
+#define ORN_DEC(M_)                                                               \
+  case M_:                                                                        \
+    if (p.mode == DRO_POSTNORM) ORN_DEC_PF(M_, PF_POSTNORM);                      \
+    if (p.mode == DRO_GATED) ORN_DEC_PF(M_, PF_GATED);                            \
+    ORN_DEC_PF(M_, PF_STREAM)
   switch (M) {
     ORN_DEC(1);
     ORN_DEC(2);
@@ -1011,5 +1023,6 @@ int f_decode_dense(orn_ctx* ctx, cudaStream_t s, int M, const DecodePrologue& p,
     ORN_DEC(4);
   }
 #undef ORN_DEC
+#undef ORN_DEC_PF
   return ORN_ERR_ARG;
 }

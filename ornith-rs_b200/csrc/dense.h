@@ -67,7 +67,7 @@ struct GroupGate {
   int ldo = 0, ldg = 0;           // multiples of 8
   int n = 0, group = 1;           // n entries, n % group == 0
   const bf16_t* w = nullptr;      // [n]
-  int act = ACT_SIGMOID;
+  int act = ACT_SIGMOID;          // or ACT_SILU
   float eps = 0.f;
 };
 int k_group_gate_rows(orn_ctx* ctx, cudaStream_t s, int rows, const GroupGate& g, void* out, int ldout, bool act_f32);
