@@ -321,7 +321,7 @@ int32_t orn_model_init_random(orn_model* m, uint64_t seed);
  * + config.json in `dir`; mtp sidecar if present */
 int32_t orn_model_load(orn_ctx* ctx, const char* dir, int32_t max_ctx, orn_model** out);
 /* The same with the activation type stated.  config.json chooses the architecture: its "architecture"
- * names an entry of the model registry ("Peratar"); without one it is the Qwen3.5-MoE trunk (bfloat16
+ * names an entry of the model registry ("Peratar", "Dokulorn"); without one it is the Qwen3.5-MoE trunk (bfloat16
  * only).  ORN_DT_F32 runs everything in true float32 (bf16 weights, float32 activations and caches). */
 #define ORN_DT_BF16 0
 #define ORN_DT_F32 1
